@@ -1,4 +1,4 @@
-"""ctypes binding of libb200kv.so (declared in include/b200kv.h).
+"""ctypes binding of libb200kv.so (include/b200kv.h) and libb200dec.so (include/b200dec.h).
 
 Loading never falls back to anything: a missing or unloadable library raises, and every
 wrapper raises on a negative return code."""
@@ -30,7 +30,22 @@ class Table(C.Structure):
     _fields_ = [("ids", c_void_p), ("stride", c_int32), ("max_pages", c_int32)]
 
 
+class DecCache(C.Structure):
+    """struct b200dec_cache"""
+
+    _fields_ = [("k", c_void_p), ("v", c_void_p), ("num_pages", c_int32), ("kv_heads", c_int32), ("page_size", c_int32),
+                ("k_dim", c_int32), ("v_dim", c_int32), ("k_row", c_int32), ("v_row", c_int32), ("elem", c_int32)]
+
+
+class DecRows(C.Structure):
+    """struct b200dec_rows"""
+
+    _fields_ = [("seq_ids", c_void_p), ("positions", c_void_p), ("cached_lens", c_void_p), ("num_decoding", c_void_p),
+                ("num_rows", c_int32)]
+
+
 P_CACHE, P_TABLE = C.POINTER(Cache), C.POINTER(Table)
+P_DCACHE, P_ROWS = C.POINTER(DecCache), C.POINTER(DecRows)
 
 # name -> (restype, argtypes); must list every function include/b200kv.h declares
 SIGNATURES = {
@@ -85,7 +100,31 @@ SIGNATURES = {
                                             c_void_p, c_int64, c_int64, c_int32, c_int32, c_int32, c_void_p, c_void_p]),
 }
 
+# entry points of libb200dec.so: every function include/b200dec.h declares, and the ones it shares with libb200kv.so
+DECODER_SIGNATURES = {
+    "b200dec_embed": (c_int32, [c_void_p, c_int32, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32, c_void_p, c_void_p]),
+    "b200dec_scaled_add_norm": (c_int32, [c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_void_p, c_float, c_float, c_void_p,
+                                          c_void_p, c_int32, c_int32, c_void_p, c_int32, c_void_p]),
+    "b200dec_rope_write": (c_int32, [c_void_p, c_int64, P_ROWS, P_DCACHE, P_TABLE, c_void_p, c_int32, c_int32, c_int32, c_int32,
+                                     c_int32, c_float, c_void_p, c_void_p, c_void_p]),
+    "b200dec_attn_rows": (c_int32, [c_void_p, P_DCACHE, P_TABLE, P_ROWS, c_int32, c_float, c_void_p, c_void_p, c_void_p]),
+    "b200dec_decode_attn_workspace": (c_size_t, [c_int32, c_int32, c_int32, c_int32, c_int32]),
+    "b200dec_decode_attn": (c_int32, [c_void_p, P_DCACHE, P_TABLE, c_void_p, c_void_p, c_int32, c_int32, c_float, c_void_p, c_int32,
+                                      c_void_p, c_size_t, c_int32, c_void_p, c_void_p]),
+    "b200dec_prefill_attn": (c_int32, [c_void_p, P_DCACHE, P_TABLE, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
+                                       c_int32, c_float, c_void_p, c_void_p, c_void_p]),
+    "b200dec_router": (c_int32, [c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p, c_void_p, c_void_p,
+                                 c_void_p]),
+    "b200dec_dispatch": (c_int32, [c_void_p, c_int32, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_int32,
+                                   c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_void_p]),
+    "b200dec_grouped_linear": (c_int32, [c_void_p, c_void_p, c_int32, c_void_p, c_int32, c_int32, c_int32, c_int32, c_int32, c_int32,
+                                         c_void_p, c_int32, c_float, c_float, c_void_p, c_int32, c_int32, c_void_p, c_void_p]),
+}
+SHARED_SIGNATURES = ("b200kv_version", "b200kv_error_string", "b200kv_set_chained_launch", "b200kv_get_chained_launch",
+                     "b200kv_sample_workspace_bytes", "b200kv_sample")
+
 _lib = None
+_decoder_lib = None
 
 
 class B200KVError(RuntimeError):
@@ -128,7 +167,26 @@ def load(build_if_needed: bool = True) -> C.CDLL:
     return lib
 
 
+def load_decoder() -> C.CDLL:
+    """Load (building first if sources are newer) libb200dec.so.  Raises if impossible."""
+    global _decoder_lib
+    if _decoder_lib is not None:
+        return _decoder_lib
+    lib = C.CDLL(_build.build_library(_build.DECODER_LIB))
+    for name in SHARED_SIGNATURES:
+        getattr(lib, name).restype, getattr(lib, name).argtypes = SIGNATURES[name]
+    for name, (res, args) in DECODER_SIGNATURES.items():
+        getattr(lib, name).restype, getattr(lib, name).argtypes = res, args
+    _decoder_lib = lib
+    return lib
+
+
+def either() -> C.CDLL:
+    """Whichever library is loaded already (the full one first), for the entry points both hold."""
+    return _lib or _decoder_lib or load()
+
+
 def check(rc: int, what: str) -> None:
     if rc != 0:
-        msg = load().b200kv_error_string(rc)
+        msg = either().b200kv_error_string(rc)
         raise ValueError(f"{what}: {msg.decode() if msg else rc}")

@@ -1,6 +1,10 @@
-"""Builds libb200kv.so (the C-ABI CUDA library) in-tree with nvcc for sm_100a.
+"""Builds the C-ABI CUDA libraries in-tree with nvcc for sm_100a.
 
     python -m inference_engine_b200.build [--force]
+
+libb200kv.so holds the int8-cache attention path and the ops around it (include/b200kv.h), libb200dec.so the decoder ops
+in the model's own precision (include/b200dec.h) with the sampler and the status words, so that serving a model of that
+kind needs the second library only.  Units are compiled side by side, and only when they changed.
 
 The write-path translation unit is compiled with -fmad=false: its results must be bit-identical
 to separately rounded IEEE fp32 arithmetic.  There is no other backend and no fallback: if the
@@ -12,6 +16,7 @@ import os
 import shutil
 import subprocess
 import sys
+from concurrent.futures import ThreadPoolExecutor
 
 PKG = os.path.dirname(os.path.abspath(__file__))
 ROOT = os.path.dirname(PKG)
@@ -22,7 +27,7 @@ OBJ_DIR = os.path.join(PKG, "build")
 
 ARCH = ["-gencode", "arch=compute_100a,code=sm_100a"]
 COMMON = ["-O3", "-lineinfo", "-std=c++17", "-Xcompiler", "-fPIC", "-I", INCLUDE, "-I", CSRC]
-UNITS = {
+UNITS = {  # unit -> extra flags
     "abi.cu": [],
     "write_kernels.cu": ["-fmad=false"],
     "decode_attn.cu": [],
@@ -31,6 +36,18 @@ UNITS = {
     "block_ops.cu": [],
     "sampler.cu": ["-fmad=false"],
     "skinny_linear_tc5.cu": [],
+    "row_ops.cu": [],
+    "paged_rows.cu": [],
+    "paged_decode.cu": [],
+    "paged_prefill_tc5.cu": [],
+    "moe.cu": [],
+    "moe_gemm_tc5.cu": [],
+}
+DECODER_LIB = os.path.join(PKG, "libb200dec.so")
+LIBRARIES = {
+    LIB: ["abi.cu", "write_kernels.cu", "decode_attn.cu", "prefill_attn.cu", "prefill_attn_tc5.cu", "block_ops.cu", "sampler.cu",
+          "skinny_linear_tc5.cu"],
+    DECODER_LIB: ["abi.cu", "sampler.cu", "paged_prefill_tc5.cu", "row_ops.cu", "paged_rows.cu", "paged_decode.cu", "moe.cu", "moe_gemm_tc5.cu"],
 }
 # The same library with per-warp timestamps compiled into the decode-attention kernel (bench.py --phases);
 # never loaded by the product path.
@@ -44,36 +61,53 @@ def _nvcc() -> str:
     raise RuntimeError("nvcc not found: libb200kv.so cannot be built")
 
 
-def sources() -> list[str]:
-    return [os.path.join(CSRC, u) for u in UNITS if os.path.exists(os.path.join(CSRC, u))]
+def headers() -> list[str]:
+    return sorted([os.path.join(d, f) for d in (CSRC, INCLUDE) for f in os.listdir(d) if f.endswith((".cuh", ".h"))])
 
 
-def needs_build() -> bool:
-    if not os.path.exists(LIB):
+def _newer(deps: list[str], target: str) -> bool:
+    if not os.path.exists(target):
         return True
-    t = os.path.getmtime(LIB)
-    deps = sources() + [os.path.join(CSRC, "common.cuh"), os.path.join(INCLUDE, "b200kv.h")]
-    return any(os.path.getmtime(d) > t for d in deps if os.path.exists(d))
+    t = os.path.getmtime(target)
+    return any(os.path.getmtime(d) > t for d in deps)
+
+
+def needs_build(lib: str = LIB) -> bool:
+    return _newer([os.path.join(CSRC, u) for u in LIBRARIES[lib]] + headers(), lib)
+
+
+def _compile(unit: str, force: bool, verbose: bool) -> str:
+    src, obj = os.path.join(CSRC, unit), os.path.join(OBJ_DIR, unit.replace(".cu", ".o"))
+    if force or _newer([src] + headers(), obj):
+        tmp = f"{obj}.{os.getpid()}"
+        cmd = [_nvcc(), *ARCH, *COMMON, *UNITS[unit], "-c", src, "-o", tmp]
+        if verbose:
+            cmd.insert(1, "-Xptxas=-v")
+        subprocess.run(cmd, check=True, stdout=sys.stderr if not verbose else None)
+        os.replace(tmp, obj)
+    return obj
+
+
+def build_library(lib: str, force: bool = False, verbose: bool = False) -> str:
+    """One library, with the units it needs and no others."""
+    if not force and not needs_build(lib):
+        return lib
+    os.makedirs(OBJ_DIR, exist_ok=True)
+    with ThreadPoolExecutor(max_workers=max(1, min(8, os.cpu_count() or 1))) as pool:
+        objs = list(pool.map(lambda u: _compile(u, force, verbose), LIBRARIES[lib]))
+    tmp = f"{lib}.{os.getpid()}"
+    subprocess.run([_nvcc(), *ARCH, "-shared", "-cudart", "static", "-o", tmp, *objs], check=True)
+    os.replace(tmp, lib)
+    return lib
 
 
 def build(force: bool = False, verbose: bool = False) -> str:
-    if not force and not needs_build():
-        return LIB
-    nvcc = _nvcc()
-    os.makedirs(OBJ_DIR, exist_ok=True)
-    objs = []
-    for unit, extra in UNITS.items():
-        src = os.path.join(CSRC, unit)
-        obj = os.path.join(OBJ_DIR, unit.replace(".cu", ".o"))
-        cmd = [nvcc, *ARCH, *COMMON, *extra, "-c", src, "-o", obj]
-        if verbose:
-            cmd.insert(1, "-Xptxas=-v")
-        subprocess.run(cmd, check=True)
-        objs.append(obj)
-    tmp = LIB + ".tmp"
-    subprocess.run([nvcc, *ARCH, "-shared", "-cudart", "static", "-o", tmp, *objs], check=True)
-    os.replace(tmp, LIB)
-    build_stamps(nvcc, objs)
+    """Every library (and the instrumented one of bench.py --phases).  Returns the path of libb200kv.so."""
+    stale = force or needs_build(LIB) or not os.path.exists(STAMPS_LIB)
+    build_library(DECODER_LIB, force, verbose)
+    build_library(LIB, force, verbose)
+    if stale:
+        build_stamps(_nvcc(), [os.path.join(OBJ_DIR, u.replace(".cu", ".o")) for u in LIBRARIES[LIB]])
     return LIB
 
 

@@ -1,0 +1,82 @@
+// Helpers shared by the b200dec kernels: element conversion, cache addressing, reductions.
+#pragma once
+#include "b200dec.h"
+#include "common.cuh"
+
+namespace b200kv {
+
+__device__ __forceinline__ float ld_elem(const uint16_t* p) { return bf16_bits_to_float(*p); }
+__device__ __forceinline__ float ld_elem(const float* p) { return *p; }
+__device__ __forceinline__ void st_elem(uint16_t* p, float v) { *p = (uint16_t)float_to_bf16_bits(v); }
+__device__ __forceinline__ void st_elem(float* p, float v) { *p = v; }
+
+// 4 consecutive elements (16-byte aligned fp32, 8-byte aligned bf16)
+__device__ __forceinline__ void ld_elem4(const float* p, float (&f)[4]) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+__device__ __forceinline__ void ld_elem4(const uint16_t* p, float (&f)[4]) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xFFFF0000u);
+  f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xFFFF0000u);
+}
+__device__ __forceinline__ void st_elem4(float* p, const float (&f)[4]) {
+  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+}
+__device__ __forceinline__ void st_elem4(uint16_t* p, const float (&f)[4]) {
+  uint2 v;
+  v.x = float_to_bf16_bits(f[0]) | (float_to_bf16_bits(f[1]) << 16);
+  v.y = float_to_bf16_bits(f[2]) | (float_to_bf16_bits(f[3]) << 16);
+  *reinterpret_cast<uint2*>(p) = v;
+}
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+
+// Device view of a b200dec_cache with its page table.
+struct DecCache {
+  void* k;
+  void* v;
+  int num_pages, heads, P, k_dim, v_dim, k_row, v_row;
+  const int32_t* table;
+  int table_stride, max_pages;
+};
+inline DecCache dec_view(const b200dec_cache* c, const b200kv_table* t) {
+  return DecCache{c->k, c->v, c->num_pages, c->kv_heads, c->page_size, c->k_dim, c->v_dim, c->k_row, c->v_row,
+                  t->ids, t->stride, t->max_pages};
+}
+// Page of token position `pos` of entry b, or -1 (with a status bit).
+__device__ __forceinline__ int dec_page(const DecCache& c, int b, int pos, int32_t* status) {
+  const int slot = pos / c.P;
+  if (pos < 0 || slot >= c.max_pages) {
+    if (status) atomicOr(status, B200KV_S_BAD_POSITION);
+    return -1;
+  }
+  const int page = c.table[(long long)b * c.table_stride + slot];
+  if (page < 0 || page >= c.num_pages) {
+    if (status) atomicOr(status, B200KV_S_BAD_PAGE);
+    return -1;
+  }
+  return page;
+}
+// First element of row `prow` of (page, head) in k / v.
+__device__ __forceinline__ long long dec_row(const DecCache& c, int page, int head, int prow) {
+  return ((long long)page * c.heads + head) * c.P + prow;
+}
+
+inline int check_dec_cache(const b200dec_cache* c, const b200kv_table* t) {
+  if (!c || !t || !c->k || !c->v || !t->ids) return B200KV_E_NULL;
+  if (c->num_pages < 1 || c->kv_heads < 1 || c->page_size < 1 || c->k_dim < 1 || c->v_dim < 1) return B200KV_E_SHAPE;
+  if (c->k_row != (c->k_dim + 7) / 8 * 8 || c->v_row != (c->v_dim + 7) / 8 * 8) return B200KV_E_SHAPE;
+  if (c->elem != 2 && c->elem != 4) return B200KV_E_SHAPE;
+  if (t->max_pages < 1 || t->stride < 0) return B200KV_E_SHAPE;
+  if (!aligned(c->k, 16) || !aligned(c->v, 16)) return B200KV_E_ALIGN;
+  return B200KV_OK;
+}
+
+inline int launch_result(cudaError_t e) { return e == cudaSuccess && cudaGetLastError() == cudaSuccess ? B200KV_OK : B200KV_E_LAUNCH; }
+
+}  // namespace b200kv

@@ -1,0 +1,247 @@
+// The paged cache of unquantised rows: rotary positions + unit norm + write of keys and values (one kernel), and the
+// general attention over it (any sizes, bf16 or fp32, prompt portions and decoding alike) on the CUDA cores.
+#include "dec_common.cuh"
+
+namespace b200kv {
+
+constexpr int kRwWarps = 8;
+constexpr int kRwMaxPairs = 16;  // a lane holds up to 32 channels: heads of up to 1024
+
+// One warp per (row, head), heads in the order q | k | v.  A lane owns channels 2 * lane + 64 * i and the next one.
+template <typename T>
+__global__ void __launch_bounds__(kRwWarps * 32)
+rope_write_kernel(const T* __restrict__ qkv, long long qkv_stride, b200dec_rows rows, DecCache c, const float* __restrict__ cos_sin,
+                  int table_len, int half, int heads, int write_kv, int unit_norm, float eps, T* __restrict__ q_out, int32_t* status) {
+  pdl_enter();
+  const int hkv = write_kv ? c.heads : 0, per_row = heads + 2 * hkv;
+  const long long item = (long long)blockIdx.x * kRwWarps + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (item >= (long long)rows.num_rows * per_row) return;
+  const int r = (int)(item / per_row), j = (int)(item - (long long)r * per_row);
+  const int kind = j < heads ? 0 : (j < heads + hkv ? 1 : 2);  // q, k, v
+  int seq = r, pos;
+  if (rows.seq_ids) {
+    seq = rows.seq_ids[r];
+    pos = rows.positions[r];
+  } else {
+    if (r >= *rows.num_decoding) {  // an idle row: nothing is written to the cache, q reads as zero
+      pdl_wait();
+      if (kind == 0)
+        for (int ch = lane; ch < c.k_row; ch += 32) st_elem(q_out + ((long long)r * heads + j) * c.k_row + ch, 0.f);
+      return;
+    }
+    pos = rows.cached_lens[r];
+  }
+  const bool ok = pos >= 0 && (half == 0 || pos < table_len);
+  if (!ok) {
+    if (lane == 0 && status) atomicOr(status, B200KV_S_BAD_POSITION);
+    pos = 0;
+  }
+  T* dst;
+  int dim = c.k_dim, row_len = c.k_row;
+  long long src_off;
+  if (kind == 0) {
+    dst = q_out + ((long long)r * heads + j) * c.k_row;
+    src_off = (long long)j * c.k_dim;
+  } else {
+    const int h = kind == 1 ? j - heads : j - heads - hkv;
+    const int page = ok ? dec_page(c, seq, pos, lane == 0 ? status : nullptr) : -1;
+    if (page < 0) return;
+    const long long at = dec_row(c, page, h, pos % c.P);
+    if (kind == 1) {
+      dst = (T*)c.k + at * c.k_row;
+      src_off = (long long)(heads + h) * c.k_dim;
+    } else {
+      dst = (T*)c.v + at * c.v_row;
+      src_off = (long long)(heads + hkv) * c.k_dim + (long long)h * c.v_dim;
+      dim = c.v_dim;
+      row_len = c.v_row;
+    }
+  }
+  pdl_wait();
+  const T* src = qkv + r * qkv_stride + src_off;
+  float y[kRwMaxPairs][2];
+  float ss = 0.f;
+  const float2* cs = reinterpret_cast<const float2*>(cos_sin) + (long long)pos * half;
+#pragma unroll
+  for (int i = 0; i < kRwMaxPairs; ++i) {
+    if (64 * i < dim) {
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int ch = 64 * i + 2 * lane + e;
+        float v = 0.f;
+        if (ch < dim) {
+          v = ld_elem(src + ch);
+          if (kind < 2 && ch < 2 * half) {
+            const bool low = ch < half;
+            const float other = ld_elem(src + (low ? ch + half : ch - half));
+            const float2 a = cs[low ? ch : ch - half];
+            v = low ? v * a.x - other * a.y : v * a.x + other * a.y;
+          }
+        }
+        y[i][e] = v;
+        ss = fmaf(v, v, ss);
+      }
+    }
+  }
+  float inv = 1.f;
+  if (kind < 2 && unit_norm) inv = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
+#pragma unroll
+  for (int i = 0; i < kRwMaxPairs; ++i) {
+    const int ch = 64 * i + 2 * lane;
+    if (ch < row_len) {  // row_len is even; channels behind dim are zero
+      if (sizeof(T) == 2)
+        *reinterpret_cast<uint32_t*>(dst + ch) = float_to_bf16_bits(y[i][0] * inv) | (float_to_bf16_bits(y[i][1] * inv) << 16);
+      else
+        *reinterpret_cast<float2*>(dst + ch) = make_float2(y[i][0] * inv, y[i][1] * inv);
+    }
+  }
+}
+
+// ---------------------------------------------------------------- attention, one block per (row, query head)
+constexpr int kArThreads = 128;
+constexpr int kArKeys = 128;  // keys per block step, one score per thread
+constexpr int kArPieces = 8;  // channels of the output per thread: v_dim up to 1024
+
+template <typename T>
+__global__ void __launch_bounds__(kArThreads)
+attn_rows_kernel(const T* __restrict__ q, DecCache c, b200dec_rows rows, int heads, float scale, T* __restrict__ out, int32_t* status) {
+  extern __shared__ float ar_smem[];
+  float* qs = ar_smem;                                                  // [k_dim]
+  float* ps = qs + ((c.k_dim + 3) / 4) * 4;                             // [kArKeys]
+  int* pages = reinterpret_cast<int*>(ps + kArKeys);                    // [kArKeys] row index of each key in the cache
+  __shared__ float red[2][kArThreads / 32];
+  pdl_enter();
+  const int r = blockIdx.y, h = blockIdx.x, hk = h / (heads / c.heads), tid = threadIdx.x;
+  T* dst = out + ((long long)r * heads + h) * c.v_dim;
+  int seq = r, pos;
+  if (rows.seq_ids) {
+    seq = rows.seq_ids[r];
+    pos = rows.positions[r];
+  } else {
+    pos = r < *rows.num_decoding ? rows.cached_lens[r] : -1;
+  }
+  pdl_wait();
+  if (pos < 0) {  // idle row
+    for (int ch = tid; ch < c.v_dim; ch += kArThreads) st_elem(dst + ch, 0.f);
+    return;
+  }
+  const T* qrow = q + ((long long)r * heads + h) * c.k_row;
+  for (int ch = tid; ch < c.k_dim; ch += kArThreads) qs[ch] = ld_elem(qrow + ch) * scale;
+  float m = -INFINITY, l = 0.f, o[kArPieces];
+#pragma unroll
+  for (int i = 0; i < kArPieces; ++i) o[i] = 0.f;
+  for (int j0 = 0; j0 <= pos; j0 += kArKeys) {
+    const int n = min(kArKeys, pos + 1 - j0);
+    __syncthreads();
+    int at = -1;
+    float s = -INFINITY;
+    if (tid < n) {
+      const int page = dec_page(c, seq, j0 + tid, status);
+      if (page >= 0) {
+        at = page * c.P + (j0 + tid) % c.P;  // token slot; head and row strides are applied below
+        const T* krow = (const T*)c.k + dec_row(c, page, hk, (j0 + tid) % c.P) * c.k_row;
+        float acc = 0.f;
+        for (int ch = 0; ch < c.k_row; ch += 4) {
+          float f[4];
+          ld_elem4(krow + ch, f);
+#pragma unroll
+          for (int e = 0; e < 4; ++e)
+            if (ch + e < c.k_dim) acc = fmaf(qs[ch + e], f[e], acc);
+        }
+        s = acc;
+      }
+    }
+    pages[tid] = at;
+    float mx = s;
+#pragma unroll
+    for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+    if ((tid & 31) == 0) red[0][tid >> 5] = mx;
+    __syncthreads();
+    mx = fmaxf(fmaxf(red[0][0], red[0][1]), fmaxf(red[0][2], red[0][3]));
+    const float mn = fmaxf(m, mx), base = mn == -INFINITY ? 0.f : mn;
+    const float p = expf(s - base), alpha = expf(m - base);
+    m = mn;
+    ps[tid] = p;
+    const float sum = warp_sum(p);
+    if ((tid & 31) == 0) red[1][tid >> 5] = sum;
+    __syncthreads();
+    l = l * alpha + (red[1][0] + red[1][1]) + (red[1][2] + red[1][3]);
+#pragma unroll
+    for (int i = 0; i < kArPieces; ++i) o[i] *= alpha;
+    for (int k = 0; k < n; ++k) {
+      const int slot = pages[k];
+      if (slot < 0) continue;
+      const int page = slot / c.P;
+      const T* vrow = (const T*)c.v + dec_row(c, page, hk, slot - page * c.P) * c.v_row;
+      const float w = ps[k];
+#pragma unroll
+      for (int i = 0; i < kArPieces; ++i) {
+        const int ch = tid + i * kArThreads;
+        if (ch < c.v_dim) o[i] = fmaf(w, ld_elem(vrow + ch), o[i]);
+      }
+    }
+  }
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+#pragma unroll
+  for (int i = 0; i < kArPieces; ++i) {
+    const int ch = tid + i * kArThreads;
+    if (ch < c.v_dim) st_elem(dst + ch, o[i] * inv);
+  }
+}
+
+}  // namespace b200kv
+
+using namespace b200kv;
+
+static int check_rows(const b200dec_rows* r) {
+  if (!r) return B200KV_E_NULL;
+  if (r->num_rows < 0) return B200KV_E_SHAPE;
+  if ((r->seq_ids == nullptr) != (r->positions == nullptr)) return B200KV_E_NULL;
+  if (!r->seq_ids && (!r->cached_lens || !r->num_decoding)) return B200KV_E_NULL;
+  return B200KV_OK;
+}
+
+extern "C" int b200dec_rope_write(const void* qkv, int64_t qkv_stride, const b200dec_rows* rows, const b200dec_cache* cache,
+                                  const b200kv_table* table, const float* cos_sin, int32_t table_len, int32_t half, int32_t heads,
+                                  int32_t write_kv, int32_t unit_norm, float eps, void* q_out, int32_t* status, void* stream) {
+  if (rows && rows->num_rows == 0) return B200KV_OK;
+  if (!qkv || !q_out) return B200KV_E_NULL;
+  int rc = check_rows(rows);
+  if (rc == B200KV_OK) rc = check_dec_cache(cache, table);
+  if (rc != B200KV_OK) return rc;
+  if (half < 0 || 2 * half > cache->k_dim || (half > 0 && (!cos_sin || table_len < 1))) return B200KV_E_SHAPE;
+  if (heads < 1 || heads % cache->kv_heads || cache->k_row > 64 * kRwMaxPairs || cache->v_row > 64 * kRwMaxPairs) return B200KV_E_SHAPE;
+  if (!aligned(q_out, 16) || !aligned(cos_sin, 8)) return B200KV_E_ALIGN;
+  const long long items = (long long)rows->num_rows * (heads + (write_kv ? 2 * cache->kv_heads : 0));
+  const long long blocks = (items + kRwWarps - 1) / kRwWarps;
+  if (blocks > 0x7FFFFFFFll) return B200KV_E_RANGE;
+  const DecCache c = dec_view(cache, table);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (cache->elem == 2)
+    return launch_result(launch_chained(rope_write_kernel<uint16_t>, dim3((unsigned)blocks), dim3(kRwWarps * 32), 0, s, (const uint16_t*)qkv,
+                                        (long long)qkv_stride, *rows, c, cos_sin, table_len, half, heads, write_kv, unit_norm, eps,
+                                        (uint16_t*)q_out, status));
+  return launch_result(launch_chained(rope_write_kernel<float>, dim3((unsigned)blocks), dim3(kRwWarps * 32), 0, s, (const float*)qkv,
+                                      (long long)qkv_stride, *rows, c, cos_sin, table_len, half, heads, write_kv, unit_norm, eps,
+                                      (float*)q_out, status));
+}
+
+extern "C" int b200dec_attn_rows(const void* q, const b200dec_cache* cache, const b200kv_table* table, const b200dec_rows* rows,
+                                 int32_t heads, float scale, void* out, int32_t* status, void* stream) {
+  if (rows && rows->num_rows == 0) return B200KV_OK;
+  if (!q || !out) return B200KV_E_NULL;
+  int rc = check_rows(rows);
+  if (rc == B200KV_OK) rc = check_dec_cache(cache, table);
+  if (rc != B200KV_OK) return rc;
+  if (heads < 1 || heads % cache->kv_heads || cache->v_dim > kArThreads * kArPieces || cache->k_dim > 1024) return B200KV_E_SHAPE;
+  if ((long long)cache->num_pages * cache->page_size > 0x7FFFFFFFll || rows->num_rows > 65535) return B200KV_E_RANGE;
+  const size_t smem = (size_t)((cache->k_dim + 3) / 4 * 4 + 2 * kArKeys) * 4;
+  const DecCache c = dec_view(cache, table);
+  cudaStream_t s = (cudaStream_t)stream;
+  if (cache->elem == 2)
+    return launch_result(launch_chained(attn_rows_kernel<uint16_t>, dim3(heads, rows->num_rows), dim3(kArThreads), smem, s,
+                                        (const uint16_t*)q, c, *rows, heads, scale, (uint16_t*)out, status));
+  return launch_result(launch_chained(attn_rows_kernel<float>, dim3(heads, rows->num_rows), dim3(kArThreads), smem, s, (const float*)q, c,
+                                      *rows, heads, scale, (float*)out, status));
+}

@@ -21,8 +21,10 @@ need are still uncommitted, so a running request can never run out.  The first p
 scratch run no request owns: padded entries of a graph replay write there.
 
 `Scheduler` is host-only (no torch, no GPU) so that the policy is testable on its own; `Engine` adds the
-device side.  The model is the random-init decoder of scaffold.py; sampling is the library's Gumbel-max sampler
-(greedy at tau = 0).
+device side.  It drives any model of the registry (models/__init__.py): the model makes its own caches and runs one
+step; sampling is the library's Gumbel-max sampler (greedy at tau = 0).  Besides generating (`submit_request`, `step`),
+the engine replays given tokens (`open_replay`, `replay`, `close_replay`) through the same step, cache and graphs and
+hands out the logits of any of them.
 """
 from __future__ import annotations
 
@@ -177,9 +179,9 @@ class Scheduler:
 
 
 class Engine:
-    """Scheduler + device execution.  `model` is a scaffold.DecoderScaffold on a CUDA device."""
+    """Scheduler + device execution.  `model`: an instance of a registered model class on a CUDA device."""
 
-    def __init__(self, model, max_batch_size: int, max_len: int, stop_token_id: int, page_size: int = 16,
+    def __init__(self, model, max_batch_size: int, max_len: int, stop_token_id: int, page_size: int | None = None,
                  num_pages: int | None = None, max_tokens_per_step: int = 1024, min_first_chunk: int = 64,
                  max_graph_tokens: int = 512, use_graphs: bool = True, block_m: int = 128, tau: float = 0.0, seed: int = 0):
         import numpy as np
@@ -190,6 +192,7 @@ class Engine:
 
         self.torch, self.K, self.S, self.np = torch, K, S, np
         self.model, self.device = model, model.device
+        page_size = model.page_size if page_size is None else page_size
         model.tau = float(tau)  # baked into the graphs at capture, like the reference's (engine.py:399)
         model.seed.fill_(seed)
         self.page_size, self.max_len, self.block_m = page_size, max_len, block_m
@@ -208,8 +211,7 @@ class Engine:
         self.pool = PagePool(num_pages, first=self.scratch_pages)
         self.sched = Scheduler(max_batch_size, max_len, page_size, self.pool, max_tokens_per_step, min_first_chunk,
                                stop_token_id)
-        self.caches = [K.make_layer_cache(num_pages, S.HKV, page_size, S.D, device=self.device)
-                       for _ in range(model.num_layers)]
+        self.caches = model.make_caches(num_pages, page_size, self.max_pages * page_size)
         # one int32 buffer per kind of step, filled on the host and copied in one piece
         cap = sum(self.mixed_layout(max_tokens_per_step))
         self.host_mixed = torch.empty(cap, dtype=torch.int32).pin_memory()
@@ -222,8 +224,7 @@ class Engine:
         self.scratch_row = self.np.zeros(self.max_pages, self.np.int32)
         self.scratch_row[: self.scratch_pages] = self.np.arange(self.scratch_pages)
         self.prefix_capacity = 2 * max_len
-        self.prefix_k = torch.empty(S.HKV, self.prefix_capacity, S.D, device=self.device, dtype=torch.bfloat16)
-        self.prefix_v = torch.empty_like(self.prefix_k)
+        self.prefix = model.make_prefix(self.prefix_capacity)  # None: the model reads its cache by page
         self.graph_pool = torch.cuda.graph_pool_handle()  # one pool for all graphs: only one runs at a time
         self.decode_graphs: dict[int, tuple] = {}
         self.mixed_graphs: dict[int, tuple] = {}
@@ -248,7 +249,7 @@ class Engine:
         if step is None:
             return []
         t1 = time.perf_counter()
-        tokens = self.run_decode(step) if step.decode_only else self.run_mixed(step)
+        tokens = self.run(step).tokens[: len(step.entries)].tolist()  # the read-back ends the step
         t2 = time.perf_counter()
         finished = self.sched.commit(step, tokens)
         for r in finished:
@@ -257,6 +258,49 @@ class Engine:
         self.seconds["run (inputs, launch, read-back)"] += t2 - t1
         self.seconds["commit"] += time.perf_counter() - t2
         return finished
+
+    # ------------------------------------------------------------------ replay of given tokens
+    def open_replay(self) -> Request:
+        """A request whose tokens the caller supplies; it holds pages like any other."""
+        r = Request(self.sched.next_id, [], 0, admitted=True)
+        self.sched.next_id += 1
+        return r
+
+    def replay(self, entries: list[tuple[Request, list[int], list[int]]]):
+        """One step of (request, its next tokens, places among them whose logits are wanted).  Returns the wanted
+        logits, fp32 [wanted, vocab], in the order of the entries; the tokens the step samples are dropped."""
+        for r, toks, want in entries:
+            if not toks or r.cached_len + len(toks) > self.max_len:
+                raise ValueError(f"{r.cached_len} + {len(toks)} tokens do not fit a request of {self.max_len}")
+            if any(not 0 <= t < self.model.vocab for t in toks) or any(not 0 <= w < len(toks) for w in want):
+                raise ValueError("a token id or a wanted place is out of range")
+        # decoding entries (one token behind cached ones) come first, as in the steps the scheduler plans
+        order = sorted(range(len(entries)), key=lambda i: not (len(entries[i][1]) == 1 and entries[i][0].cached_len > 0))
+        decoding = sum(len(toks) == 1 and r.cached_len > 0 for r, toks, _ in entries)
+        for r, toks, _ in entries:
+            need = math.ceil((r.cached_len + len(toks)) / self.page_size) - len(r.pages)
+            if not self.pool.commit(need):
+                raise RuntimeError("the page pool is exhausted")
+            r.pages.extend(self.pool.take() for _ in range(need))
+        step = Step([entries[i][:2] for i in order], decoding)
+        out = self.run(step)
+        first, at = {}, 0
+        for i in order:
+            first[i] = at
+            at += len(entries[i][1])
+        rows = [first[i] + w for i, (_, _, want) in enumerate(entries) for w in want]
+        for r, toks, _ in entries:
+            r.cached_len += len(toks)
+        with self.torch.inference_mode():
+            if not rows:
+                self.torch.cuda.synchronize()
+                return self.torch.empty(0, self.model.vocab)
+            return self.model.logits(out.hidden[self.torch.tensor(rows, device=self.device)]).float().cpu()
+
+    def close_replay(self, r: Request) -> None:
+        self.pool.release(r.pages)
+        r.pages = []
+        self.rows.pop(r.id, None)
 
     # ------------------------------------------------------------------ input buffers
     def mixed_layout(self, n_tokens: int) -> list[int]:
@@ -312,10 +356,10 @@ class Engine:
         inp = S.StepInputs(ids=v[0], positions=v[1], seq_ids=v[2], cu_seqlens=v[3], cached_lens=v[4], cu_cached=v[5],
                            tile_start=v[6], num_decoding=v[7], block_table=v[8].view(self.num_entries, self.max_pages),
                            prefix_tokens=prefix_tokens, block_m=self.block_m)
-        pk, pv = self.prefix_k, self.prefix_v
-        if prefix_tokens > self.prefix_capacity:  # a one-off buffer for this step
-            pk = self.torch.empty(S.HKV, prefix_tokens, S.D, device=self.device, dtype=pk.dtype)
-            pv = self.torch.empty_like(pk)
+        if self.prefix is None:
+            return inp, None
+        # a step whose cached prefixes exceed the scratch gets a one-off buffer
+        pk, pv = self.prefix if prefix_tokens <= self.prefix_capacity else self.model.make_prefix(prefix_tokens)
         return inp, S.PrefixScratch(pk, pv, inp.cu_cached)
 
     def decode_views(self, b: int):
@@ -326,14 +370,14 @@ class Engine:
     # ------------------------------------------------------------------ execution
     def forward_mixed(self, n_pad: int, prefix_tokens: int = 0):
         inp, prefix = self.mixed_views(n_pad, prefix_tokens)
-        return self.model.forward(self.caches, inp, inp.ids, inp.cached_lens, inp.block_table, inp.num_decoding, prefix)
+        return self.model.step(self.caches, inp, inp.ids, inp.cached_lens, inp.block_table, inp.num_decoding, prefix)
 
     def forward_decode(self, b: int):
         ids, cached, nd, table = self.decode_views(b)
-        return self.model.forward(self.caches, None, ids, cached, table, nd)
+        return self.model.step(self.caches, None, ids, cached, table, nd)
 
     def capture_graph(self, run):
-        """Two eager runs first (engine.py:432-449), then the recording; returns (graph, output tensor)."""
+        """Two eager runs first (engine.py:432-449), then the recording; returns (graph, the step's output)."""
         torch = self.torch
         s = torch.cuda.Stream(device=self.device)
         s.wait_stream(torch.cuda.current_stream())
@@ -363,7 +407,11 @@ class Engine:
         if bits:
             raise RuntimeError(f"device status word {bits:#x} set while the step graphs were captured")
 
-    def run_decode(self, step: Step) -> list[int]:
+    def run(self, step: Step):
+        """Execute a planned step; the outputs' first entries / rows are the step's own."""
+        return self.run_decode(step) if step.decode_only else self.run_mixed(step)
+
+    def run_decode(self, step: Step):
         torch = self.torch
         t_in = time.perf_counter()
         B = len(step.entries)
@@ -388,16 +436,16 @@ class Engine:
             with torch.inference_mode():
                 out = self.forward_decode(b)
             self.steps_run["eager"] += 1
-        return out[:B].tolist()  # the read-back ends the step
+        return out
 
-    def run_mixed(self, step: Step) -> list[int]:
+    def run_mixed(self, step: Step):
         torch = self.torch
         N = step.num_tokens
         n_pad = next((x for x in self.token_buckets if x >= N), N)
         t_in = time.perf_counter()
         prefix_tokens = self.fill_mixed(step, n_pad)
         self.seconds["inputs"] += time.perf_counter() - t_in
-        if n_pad in self.mixed_graphs and prefix_tokens <= self.prefix_capacity:
+        if n_pad in self.mixed_graphs and (self.prefix is None or prefix_tokens <= self.prefix_capacity):
             g, out = self.mixed_graphs[n_pad]
             g.replay()
             self.steps_run["mixed_graph"] += 1
@@ -405,4 +453,4 @@ class Engine:
             with torch.inference_mode():
                 out = self.forward_mixed(n_pad, prefix_tokens)
             self.steps_run["eager"] += 1
-        return out[: len(step.entries)].tolist()
+        return out

@@ -93,6 +93,8 @@ def set_early_start(enabled: bool) -> None:
     global _early_start
     _early_start = bool(enabled)
     _lib.load().b200kv_set_chained_launch(1 if enabled else 0)
+    if _lib._decoder_lib is not None:
+        _lib._decoder_lib.b200kv_set_chained_launch(1 if enabled else 0)
 
 
 _workspaces: dict[tuple, torch.Tensor] = {}
@@ -500,7 +502,7 @@ def sample(logits: torch.Tensor, tau: float, seed: torch.Tensor) -> torch.Tensor
     assert logits.dim() == 2 and logits.stride(-1) == 1, "kernel assumes contiguous vocab dim"
     assert logits.dtype in (torch.bfloat16, torch.float32) and seed.dtype == torch.int64
     B, V = logits.shape
-    lib = _lib.load()
+    lib = _lib.either()
     nbytes = lib.b200kv_sample_workspace_bytes(B, V)
     ws = torch.empty(max(nbytes, 8), dtype=torch.uint8, device=logits.device)
     out = torch.empty(B, 1, dtype=torch.int64, device=logits.device)
@@ -539,9 +541,12 @@ def skinny_supported(M: int, N: int, K: int) -> list[int]:
     return [s for s in (1, 2, 4, 8) if s <= T // 2 and s <= K // 64]
 
 
-def linear(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:  # kernels.py:1465
+def linear(x: torch.Tensor, weight: torch.Tensor, out_dtype: torch.dtype | None = None) -> torch.Tensor:  # kernels.py:1465
     """[M, K] @ [N, K].T -> [M, N] with whichever of skinny_matmul and cuBLAS (F.linear) tune_linear measured faster
-    for this (weight shape, row count); unmeasured shapes go to cuBLAS."""
+    for this (weight shape, row count); unmeasured shapes go to cuBLAS.  `out_dtype` float32 keeps the 32-bit
+    accumulator of a bf16 product (cuBLAS only)."""
+    if out_dtype is not None and out_dtype != x.dtype:
+        return torch.mm(x, weight.t(), out_dtype=out_dtype)
     if x.dim() == 2 and x.stride(-1) == 1 and weight.stride(-1) == 1:
         s = use_skinny.get((weight.shape[0], weight.shape[1], x.shape[0]), 0)
         if s:

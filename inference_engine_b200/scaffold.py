@@ -28,6 +28,7 @@ from dataclasses import dataclass
 import torch
 
 from . import kernels as K
+from .models import StepOutput, register
 
 HIDDEN, FFN, VOCAB, LAYERS = 2048, 6144, 151936, 28
 HQ, HKV, D = 16, 8, 128
@@ -162,6 +163,7 @@ def attention_ops(q, k, v, qw, kw, cos, sin, cache, inp: StepInputs | None, cach
     return out
 
 
+@register("DecoderScaffold")
 class DecoderScaffold:
     """Weights of a Qwen3-shaped decoder, ~N(0, std), norm weights 1, tied embeddings
     (architecture.py:478-516 for the 1.7B geometry).  Not an nn.Module: inference only."""
@@ -190,6 +192,25 @@ class DecoderScaffold:
         self.seed = torch.zeros(1, dtype=torch.int64, device=device)
         self.inv_freq = ROPE_BASE ** (-torch.arange(0, D, 2, dtype=torch.float32, device=device) / D)
 
+    page_size = 16  # the engine's default for this model
+
+    @classmethod
+    def from_config(cls, config: dict, weights, device, dtype: torch.dtype = torch.bfloat16) -> "DecoderScaffold":
+        """Sizes hidden, ffn, vocab, layers (and std, seed) from the configuration; the weights are random."""
+        if weights is not None:
+            raise ValueError("DecoderScaffold has random weights only")
+        if dtype != torch.bfloat16:
+            raise ValueError("DecoderScaffold runs in bfloat16 over an int8 cache")
+        return cls(device, **{k: config[k] for k in ("hidden", "ffn", "vocab", "layers", "std", "seed") if k in config})
+
+    def make_caches(self, num_pages: int, page_size: int, max_len: int) -> list[K.LayerKVCache]:
+        return [K.make_layer_cache(num_pages, HKV, page_size, D, device=self.device) for _ in range(self.num_layers)]
+
+    def make_prefix(self, capacity: int) -> tuple[torch.Tensor, torch.Tensor]:
+        """bf16 scratch for the prefilling entries' cached tokens."""
+        k = torch.empty(HKV, capacity, D, device=self.device, dtype=torch.bfloat16)
+        return k, torch.empty_like(k)
+
     def rope(self, positions: torch.Tensor):
         ang = positions[:, None, None] * self.inv_freq[None, None, :]  # architecture.py:387-390
         return ang.cos().to(torch.bfloat16), ang.sin().to(torch.bfloat16)
@@ -199,6 +220,11 @@ class DecoderScaffold:
                 prefix: PrefixScratch | None = None):
         """One step: token ids [N] -> sampled next token per entry [entries] (int64; greedy while tau = 0).
         `inp is None` = pure decode (ids has one token per entry, position = cached length)."""
+        return self.step(caches, inp, ids, cached_lens, slot_ids, num_decoding, prefix).tokens
+
+    @torch.inference_mode()
+    def step(self, caches, inp: StepInputs | None, ids, cached_lens, slot_ids, num_decoding,
+             prefix: PrefixScratch | None = None) -> StepOutput:
         # the decode-attention work split of this step, once for all layers (it depends on the step's metadata only)
         plan = K.plan_decode_step(cached_lens, slot_ids, num_decoding, caches[0]) if self.plan_steps else None
         x = self.embed[ids.long()]
@@ -217,8 +243,11 @@ class DecoderScaffold:
             attn = K.linear(out.view(N, HQ * D), L["o"])
             residual, normed = K.add_rms_norm(residual, attn, L["ln2"], EPS)
             x = K.linear(K.silu_mul(K.linear(normed, L["gate_up"])), L["down"])
-        _, x = K.add_rms_norm(residual, x, self.norm, EPS)
+        _, hidden = K.add_rms_norm(residual, x, self.norm, EPS)
+        x = hidden
         if inp is not None:
             x = x[(inp.cu_seqlens[1:] - 1).long()]  # each entry's last row; junk for entries without tokens
-        logits = K.linear(x, self.embed)
-        return K.sample(logits, self.tau, self.seed).view(-1)
+        return StepOutput(K.sample(self.logits(x), self.tau, self.seed).view(-1), hidden)
+
+    def logits(self, hidden: torch.Tensor) -> torch.Tensor:
+        return K.linear(hidden, self.embed)
