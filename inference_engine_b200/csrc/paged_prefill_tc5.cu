@@ -26,13 +26,13 @@ extern "C" int b200dec_prefill_attn(const void* q, const b200dec_cache* cache, c
   if (!dt_cache_map(&tm_k, pg.c.k, pg.c.k_dim, pg.c.k_row, pg.c.P, ph, pg.box_rows) ||
       !dt_cache_map(&tm_v, pg.c.v, pg.c.v_dim, pg.c.v_row, pg.c.P, ph, pg.box_rows))
     return B200KV_E_LAUNCH;
+  auto kernel = pg.c.k_dim > 64 ? prefill_attn_tc5_kernel<true, 2> : prefill_attn_tc5_kernel<true, 1>;
   // the opt-in is a per-device attribute of the function: set it on every call (it is cheap)
-  if (cudaFuncSetAttribute(prefill_attn_tc5_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kT5Smem) != cudaSuccess)
-    return B200KV_E_LAUNCH;
+  if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kT5Smem) != cudaSuccess) return B200KV_E_LAUNCH;
   const uint16_t* none = nullptr;
   const int32_t* no_lens = nullptr;
   return launch_result(launch_chained(
-      prefill_attn_tc5_kernel<true>, dim3(heads, num_tiles * subs), dim3(kT5Threads), kT5Smem, (cudaStream_t)stream, (const uint16_t*)q,
+      kernel, dim3(heads, num_tiles * subs), dim3(kT5Threads), kT5Smem, (cudaStream_t)stream, (const uint16_t*)q,
       (long long)heads * pg.c.k_row, (long long)pg.c.k_row, none, 0LL, 0LL, none, 0LL, 0LL, seq_ids, cu_seqlens, tile_start, block_m, subs, none,
       none, 0LL, 0LL, no_lens, (uint16_t*)out, (long long)heads * pg.c.v_dim, (long long)pg.c.v_dim, num_rows, heads / pg.c.heads,
       scale * 1.4426950408889634f, status, tm_k, tm_v, tm_k, tm_v, 0, 0, pg));

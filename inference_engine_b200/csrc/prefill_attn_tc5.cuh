@@ -42,7 +42,7 @@
 // The kernel has two forms.  The dense one (kPaged = false, prefill_attn_tc5.cu) attends [prefix | own chunk] as above with
 // head size 128.  The paged one (kPaged = true, paged_prefill_tc5.cu) reads keys and values of the whole sequence, the
 // chunk's own included, by page from a cache of bf16 rows, with key and value sizes of up to 128 each: copies beyond a
-// size read as zero, products run over the channels there are, and a query at position p sees keys 0..p.
+// size read as zero, products run over the blocks of 64 channels there are, and a query at position p sees keys 0..p.
 //
 // Every wait on an mbarrier is bounded: if a completion never arrives the waiting role records it, stops
 // issuing work and the CTA skips its stores, sets B200KV_S_TIMEOUT in the status word, frees its tensor
@@ -178,7 +178,7 @@ struct T5Paged {
   int box_rows;
 };
 
-template <bool kPaged>
+template <bool kPaged, int kKeyBlocks = 2>  // kKeyBlocks: 64-channel blocks of a key (2 covers up to 128 channels)
 __global__ void __launch_bounds__(kT5Threads, 1)
 prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long long q_sh, const uint16_t* __restrict__ k,
                         long long k_sn, long long k_sh, const uint16_t* __restrict__ v, long long v_sn, long long v_sh,
@@ -208,7 +208,7 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
   // a step in which no entry has a cached prefix may pass empty prefix tensors (no storage: NULL pointers)
   const int prefix_start = kPaged ? 0 : cu_cached[seq], prefix_len = (!kPaged && k_prefix && v_prefix) ? cu_cached[seq + 1] - prefix_start : 0;
   const int cached = kPaged ? pg.cached_lens[seq] : 0;  // keys in front of the chunk's first row, in the same list
-  const int kdim = kPaged ? pg.c.k_dim : kD, vdim = kPaged ? pg.c.v_dim : kD;
+  const int vdim = kPaged ? pg.c.v_dim : kD;
   const int seq_start = cu_seqlens[seq], seq_end = min(cu_seqlens[seq + 1], N);
   const int row_end = min(tile_row + block_m, seq_end);
   const int row0 = tile_row + sub * kT5Tile;  // first query row of this CTA
@@ -302,7 +302,7 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
         // the product that read this slot three blocks ago has completed
         if (h >= 3 && !t5_mbar_wait(empty, (h / 3 - 1) & 1, spin)) { live = false; break; }
         if constexpr (kPaged) {
-          const int dim = is_v ? vdim : kdim, blocks = dim > 64 ? 2 : 1;
+          const int blocks = is_v ? (vdim > 64 ? 2 : 1) : kKeyBlocks;
           if (!is_v || count == kT5Keys) {
             // keys behind the last one may be anything: their scores are never looked at
             if (lane == 0) {
@@ -366,7 +366,6 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
       const uint64_t dq = t5_desc(sQ, 16, 1024), dk = t5_desc(ring_k(w), 16, 1024);
       const uint64_t dv = t5_desc(ring_v(w), kT5Keys * 128, 1024);
       const uint32_t tw = tmem + 256 * w;
-      const int ksteps = kPaged ? (kdim + 15) / 16 : 8;
       const uint32_t idesc_pv = kPaged ? t5_idesc((uint32_t)((vdim + 15) / 16 * 16)) | (1u << 16) : kT5IdescPV;
       bool live = t5_mbar_wait(bar_q, 0, spin);
       auto issue_s = [&](int h) {  // S(h) = Q K(h)^T into S buffer h & 1, then the arrivals
@@ -375,8 +374,8 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
         const uint64_t kd = dk + (uint64_t)(sl * (kT5KvBytes >> 4));
         const uint32_t d = tw + 64 * (h & 1);
 #pragma unroll
-        for (int j = 0; j < 8; ++j)  // 16 channels per instruction
-          if (!kPaged || j < ksteps) t5_mma_ss(d, dq + (uint64_t)(((j >> 2) * (kT5Tile * 128) + (j & 3) * 32) >> 4),
+        for (int j = 0; j < 4 * kKeyBlocks; ++j)  // 16 channels per instruction
+          t5_mma_ss(d, dq + (uint64_t)(((j >> 2) * (kT5Tile * 128) + (j & 3) * 32) >> 4),
                     kd + (uint64_t)(((j >> 2) * (kT5Keys * 128) + (j & 3) * 32) >> 4), kT5IdescQK, j > 0);
         t5_mma_commit(bar_s(w, h & 1));
         t5_mma_commit(bar_ke(w, sl));

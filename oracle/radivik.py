@@ -93,8 +93,16 @@ def route(h, router, top):
     return ids, np.take_along_axis(s, ids, axis=1)
 
 
-def mixture(h, w, p, mlp):
+def margin(h, router, top):
+    """How far apart the last chosen and the first unchosen score of every token are (infinite without the latter)."""
+    s = np.sort(1.0 / (1.0 + np.exp(-(h @ router.T))), axis=1)
+    return s[:, -top] - s[:, -top - 1] if top < s.shape[1] else np.full(len(h), np.inf)
+
+
+def mixture(h, w, p, mlp, margins=None):
     ids, s = route(h, w[p + "router"], mlp["router"]["top"])
+    if margins is not None:
+        margins.append(margin(h, w[p + "router"], mlp["router"]["top"]))
     out = np.zeros_like(h)
     for e in range(mlp["router"]["experts"]):
         t, slot = np.nonzero(ids == e)
@@ -103,8 +111,8 @@ def mixture(h, w, p, mlp):
     return out
 
 
-def forward(cfg, w, tokens, dtype=np.float64):
-    """(logits [T, vocab], residual stream after every layer [layers, T, width])."""
+def forward(cfg, w, tokens, dtype=np.float64, margins=None):
+    """(logits [T, vocab], residual stream after every layer [layers, T, width]).  `margins`: receives every router's."""
     w = {k: np.asarray(v, dtype) for k, v in w.items()}
     eps, alpha = cfg["norm"]["eps"], cfg["postln_alpha"]
     positions = np.arange(len(tokens))
@@ -118,6 +126,6 @@ def forward(cfg, w, tokens, dtype=np.float64):
         kv = kvs[i if src is None else src]
         x = rms_norm(alpha * x + attention(x, w, p + "mix.", mx, positions, eps, kv), eps, w[p + "norm1"])
         if layer.get("mlp"):
-            x = rms_norm(alpha * x + mixture(x, w, p + "mlp.", layer["mlp"]), eps, w[p + "norm2"])
+            x = rms_norm(alpha * x + mixture(x, w, p + "mlp.", layer["mlp"], margins), eps, w[p + "norm2"])
         after.append(x)
     return rms_norm(x, eps, w["final.norm"]) @ w["head"].T, np.stack(after)

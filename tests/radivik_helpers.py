@@ -126,6 +126,21 @@ def oracle_logits(cfg, w, tokens):
     return R.forward(cfg, w, tokens)[0]
 
 
+def settle(cfg, w, tokens, least=0.01):
+    """The prompt with tokens exchanged until no router is within `least` of choosing otherwise, so that rounding cannot turn
+    a choice (two experts' outputs have nothing in common, and one turned choice would hide everything else)."""
+    tokens, g = list(tokens), np.random.default_rng(len(tokens))
+    for _ in range(600):
+        margins = []
+        R.forward(cfg, w, tokens, margins=margins)
+        close = np.nonzero(np.min(margins, axis=0) < least)[0] if margins else []
+        if len(close) == 0:
+            return tokens
+        for at in close[:3]:
+            tokens[at] = int(g.integers(0, cfg["vocab"]))
+    raise AssertionError("no settled prompt found")
+
+
 def status_clear():
     from inference_engine_b200 import kernels as K
 

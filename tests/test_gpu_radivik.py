@@ -47,7 +47,7 @@ def test_prompts_portions_and_decoding(name, dtype):
     cfg = CONFIGS[name]
     w = H.weights(cfg, 1, match=name != "small")
     eng = H.engine(H.model(cfg, w, dtype), page_size=64 if name == "sharp" else 16)
-    tokens = far_prompt(150, cfg["vocab"], 2)
+    tokens = H.settle(cfg, w, far_prompt(150, cfg["vocab"], 2))
     want = H.oracle_logits(cfg, w, tokens)
     for cuts in ([], range(1, 150), [2, 4, 7, 64, 65, 130, 132], [17, 80, 96, 128, 129], [149]):
         assert H.error(H.feed(eng, tokens, cuts), want).max() < H.TOLERANCE[dtype], cuts
@@ -59,7 +59,7 @@ def test_residual_after_every_layer(dtype):
     cfg = CONFIGS["small"]
     w = H.weights(cfg, 3)
     eng = H.engine(H.model(cfg, w, dtype))
-    tokens = prompt(23, cfg["vocab"])
+    tokens = H.settle(cfg, w, prompt(23, cfg["vocab"]))
     want = R.forward(cfg, w, tokens)[1]
     r = eng.open_replay()
     r.pages = [eng.pool.free.pop() for _ in range(2)]
@@ -81,7 +81,7 @@ def test_batches_against_each_alone(dtype):
     w = H.weights(cfg, 4, match=True)
     m = H.model(cfg, w, dtype)
     eng = H.engine(m, graphs=True)
-    reqs = [far_prompt(n, cfg["vocab"], n) for n in (97, 33, 64, 5)]
+    reqs = [H.settle(cfg, w, far_prompt(n, cfg["vocab"], n)) for n in (97, 33, 64, 5)]
     want = [H.oracle_logits(cfg, w, p) for p in reqs]
     live, at, got = [eng.open_replay() for _ in reqs], [0] * 4, [[] for _ in reqs]
     plan = [[60, 3, 0, 0], [2, 1, 64, 0], [1, 1, 0, 5], [1, 20, 0, 0], [33, 8, 0, 0]]
@@ -106,8 +106,8 @@ def test_pages_freed_and_used_again(dtype):
     w = H.weights(cfg, 5)
     eng = H.engine(H.model(cfg, w, dtype), num_pages=32 + 12, max_len=192)
     for seed, n in enumerate((150, 40, 191, 3, 100)):
-        tokens = prompt(n, cfg["vocab"], seed)
-        got = H.feed(eng, tokens, [n // 3, n // 3 + 2, n - 5, n - 4, n - 3])
+        tokens = H.settle(cfg, w, prompt(n, cfg["vocab"], seed))
+        got = H.feed(eng, tokens, sorted({max(1, c) for c in (n // 3, n // 3 + 2, n - 5, n - 4, n - 3)}))
         assert H.error(got, H.oracle_logits(cfg, w, tokens)).max() < H.TOLERANCE[dtype]
         for c in eng.caches:
             if c is not None:
@@ -126,7 +126,7 @@ def test_layers_on_another_layers_cache_hold_none():
 def test_long_decoding_with_graphs():
     cfg = CONFIGS["sharp"]
     w = H.weights(cfg, 6, match=True)
-    tokens = far_prompt(420, cfg["vocab"], 9)
+    tokens = H.settle(cfg, w, far_prompt(420, cfg["vocab"], 9))
     want = H.oracle_logits(cfg, w, tokens)
     for dtype in DTYPES:
         eng = H.engine(H.model(cfg, w, dtype), graphs=True, max_len=448)
