@@ -881,6 +881,299 @@ def run_prefill(args):
         print(json.dumps({"case": "prefill_attention", "prior_context": prior, "max_abs_diff_between_kernels": diff}), flush=True)
 
 
+def run_radivik(args):
+    """--radivik: the Radivik decoder beside the DecoderScaffold at equal size (random weights).
+
+    (1) every kernel of the new design and the like kernel of the scaffold, as fractions of their rooflines: algorithmic
+    bytes over the measured copy bandwidth or FLOPs over the measured bf16 GEMM rate, whichever takes longer; calls
+    captured in one CUDA graph over as many distinct inputs as exceed L2, median of `steps` replays;
+    (2) model steps through the registry's classes: a 1024-token prompt portion on 3072 cached tokens, and a pure decode
+    step of 64 entries with 4096 tokens each."""
+    import torch
+
+    from inference_engine_b200 import kernels as K
+    from inference_engine_b200 import ops
+    from inference_engine_b200 import scaffold as S
+    from inference_engine_b200.models import model_class
+    from inference_engine_b200.models.radivik import GATE_SLOPE
+
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    K.set_early_start(not args.no_early_start)
+    hbm = peaks()[0] * 1e9
+    tf = 1590.0
+    if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
+        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+            tf = float(json.load(f)["bf16_tflops"])
+    tf *= 1e12
+    L2 = 160e6
+    gen = torch.Generator(device=dev).manual_seed(6)
+
+    def rnd(*shape, dtype=torch.bfloat16):
+        return torch.randn(*shape, generator=gen, device=dev).to(dtype)
+
+    def i32(x):
+        return torch.tensor(x, dtype=torch.int32, device=dev)
+
+    def graph_us(calls):
+        with torch.inference_mode():
+            for _ in range(2):
+                for c in calls:
+                    c()
+            torch.cuda.synchronize()
+            g = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(g):
+                for c in calls:
+                    c()
+        for _ in range(max(args.warmup, 3)):
+            g.replay()
+        torch.cuda.synchronize()
+        ts = []
+        for _ in range(args.steps):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            g.replay()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1) * 1e3 / len(calls))
+        return statistics.median(ts)
+
+    def report(group, model, kernel, calls, nbytes, flops=0.0):
+        us = graph_us(calls)
+        roof = max(nbytes / hbm, flops / tf) * 1e6
+        print(json.dumps({"group": group, "model": model, "kernel": kernel, "us": round(us, 2), "roofline_us": round(roof, 2),
+                          "of_roofline": round(roof / us, 3), "gbs": round(nbytes / us / 1e3), "tflops": round(flops / us / 1e6, 1),
+                          "status": K.check_status(dev)}), flush=True)
+
+    def sets(nbytes):
+        return max(2, min(24, math.ceil(L2 / nbytes)))
+
+    W, FF = S.HIDDEN, S.FFN
+    sizes = {  # name: heads, kv heads, key size, value size, rotated channels, experts, top, ff
+        "as the scaffold": (16, 8, 128, 128, 128, 8, 2, FF // 2),
+        "smaller heads, more experts": (16, 8, 112, 96, 32, 32, 4, FF // 4),
+    }
+    page_r = 64
+
+    def config(sz, layers, vocab):
+        h, kv, d, vd, rot, e, top, ff = sz
+        layer = {"type": "attention", "mixer": {"heads": h, "kv_heads": kv, "dim": d, "vdim": vd, "scale": d ** -0.5,
+                                                "rot": {"dims": rot, "base": 1e6}},
+                 "mlp": {"kind": "moe", "expert": {"ff": ff, "limit": 7.0}, "router": {"experts": e, "top": top}}}
+        return {"architecture": "Radivik", "vocab": vocab, "width": W, "postln_alpha": 2.0, "norm": {"eps": 1e-6}, "layers": [layer] * layers}
+
+    # ------------------------------------------------------------------ attention and the cache write
+    def prefill_case(prior, chunk):
+        group = f"prefill attention, {chunk} rows on {prior}"
+        plan = S.plan_step([], [(prior, chunk)], chunk, 2)
+        pairs = chunk * prior + chunk * (chunk + 1) // 2
+        n = prior + chunk
+        nb = 2 * n * HKV * D * 2
+        inp = S.upload_step(plan, S.assign_pages(plan, PAGE, n // PAGE + 1)[0], [0] * chunk, dev)
+        data = [[rnd(chunk, h, D) for h in (HQ, HKV, HKV)] + [rnd(HKV, max(prior, 16), D) for _ in range(2)] for _ in range(sets(nb))]
+        report(group, "scaffold", "prefill_attention (dense prefix)",
+               [lambda d=d: K.prefill_attention(*d[:3], inp.seq_ids, inp.cu_seqlens, inp.tile_start, *d[3:], inp.cu_cached, 128) for d in data],
+               nb + 2 * chunk * HQ * D * 2, 4.0 * D * pairs * HQ)
+        for name, (h, kv, kd, vd, rot, *_) in sizes.items():
+            table, pages = S.assign_pages(plan, page_r, n // page_r + 1)
+            inp_r = S.upload_step(plan, table, [0] * chunk, dev)
+            rows = ops.Rows(chunk, inp_r.cached_lens, inp_r.num_decoding, inp_r.block_table, inp_r.seq_ids, inp_r.positions,
+                            inp_r.cu_seqlens, inp_r.tile_start, 128)
+            caches = [ops.make_paged_kv(pages, kv, page_r, kd, vd, torch.bfloat16, dev) for _ in range(sets(nb))]
+            for c in caches:
+                c.k.normal_(generator=gen)
+                c.v.normal_(generator=gen)
+            q, out = rnd(chunk, h, kd), torch.empty(chunk, h, vd, dtype=torch.bfloat16, device=dev)
+            report(group, f"Radivik, {name}", "paged_prefill_attention",
+                   [lambda c=c: ops.paged_prefill_attention(q, c, rows, kd ** -0.5, out) for c in caches],
+                   n * kv * (kd + vd) * 2 + chunk * h * (kd + vd) * 2, 2.0 * (kd + vd) * pairs * h)
+            del caches
+
+    def decode_case(B, ctx):
+        group = f"decode attention, {B} entries of {ctx}"
+        P = (ctx + PAGE - 1) // PAGE
+        cached, nd = i32([ctx - 1] * B), i32([B])
+        table = torch.randperm(B * P, generator=gen, device=dev).to(torch.int32).view(B, P)
+        nb = attn_bytes(B, ctx)
+        caches = [K.make_layer_cache(B * P, HKV, PAGE, D, device=dev) for _ in range(sets(nb))]
+        for c in caches:
+            c.k.random_(-127, 128, generator=gen)
+            c.v.random_(-127, 128, generator=gen)
+            c.k_scale.fill_(0.02)
+            c.v_scale.fill_(0.02)
+        q = rnd(B, HQ, D)
+        step_plan = K.plan_decode_step(cached, table, nd, caches[0])
+        report(group, "scaffold", "decode_attention (int8 cache)",
+               [lambda c=c: K.decode_attention(q, c, cached, table, nd, D ** -0.5, plan=step_plan) for c in caches], nb)
+        del caches
+        for name, (h, kv, kd, vd, rot, *_) in sizes.items():
+            P = (ctx + page_r - 1) // page_r
+            table_r = torch.randperm(B * P, generator=gen, device=dev).to(torch.int32).view(B, P)
+            nb = B * ctx * kv * (kd + vd) * 2 + B * h * (kd + vd) * 2
+            caches = [ops.make_paged_kv(B * P, kv, page_r, kd, vd, torch.bfloat16, dev) for _ in range(sets(nb))]
+            for c in caches:
+                c.k.normal_(generator=gen)
+                c.v.normal_(generator=gen)
+            rows = ops.Rows(B, cached, nd, table_r)
+            qr, out = rnd(B, h, kd), torch.empty(B, h, vd, dtype=torch.bfloat16, device=dev)
+            report(group, f"Radivik, {name}", "paged_decode_attention",
+                   [lambda c=c: ops.paged_decode_attention(qr, c, rows, kd ** -0.5, out, True) for c in caches], nb)
+            del caches
+
+    def write_case(N, decode):
+        group = f"rotation and cache write, {N} rows" + (" (decode)" if decode else "")
+        ctx = 512
+        plan = S.plan_step([ctx] * N, [], N, N + 1) if decode else S.plan_step([], [(ctx, N)], N, 2)
+        eps, qw = 1e-6, torch.ones(D, device=dev, dtype=torch.bfloat16)
+        table, pages = S.assign_pages(plan, PAGE, (ctx + N) // PAGE + 1)
+        inp = S.upload_step(plan, table, [0] * N, dev)
+        nb = N * ((HQ + 2 * HKV) * D * 2 + HQ * D * 2 + 2112)
+        k_sets = sets(nb)
+        caches = [K.make_layer_cache(pages, HKV, PAGE, D, device=dev) for _ in range(k_sets)]
+        qkv = [rnd(N, (HQ + 2 * HKV) * D) for _ in range(k_sets)]
+        cos, sin = rnd(N, 1, D // 2), rnd(N, 1, D // 2)
+
+        def split(t):
+            a, b, c = t.split([HQ * D, HKV * D, HKV * D], dim=-1)
+            return a.view(N, HQ, D), b.view(N, HKV, D), c.view(N, HKV, D)
+
+        if decode:
+            calls = [lambda t=t, c=c: K.fused_rope_kv_decode(*split(t), qw, qw, cos, sin, inp.block_table[:N], c, inp.cached_lens[:N],
+                                                             inp.num_decoding, eps) for t, c in zip(qkv, caches)]
+        else:
+            calls = [lambda t=t, c=c: K.write_prefill(*split(t), qw, qw, cos, sin, inp.cu_seqlens, inp.block_table, inp.cached_lens,
+                                                      inp.num_decoding, c, eps) for t, c in zip(qkv, caches)]
+        report(group, "scaffold", "fused_rope_kv_decode" if decode else "write_prefill", calls, nb)
+        for name, (h, kv, kd, vd, rot, *_) in sizes.items():
+            table, pages = S.assign_pages(plan, page_r, (ctx + N) // page_r + 1)
+            inp_r = S.upload_step(plan, table, [0] * N, dev)
+            rows = ops.Rows(N, inp_r.cached_lens, inp_r.num_decoding, inp_r.block_table)
+            if not decode:
+                rows = ops.Rows(N, inp_r.cached_lens, inp_r.num_decoding, inp_r.block_table, inp_r.seq_ids, inp_r.positions)
+            caches = [ops.make_paged_kv(pages, kv, page_r, kd, vd, torch.bfloat16, dev) for _ in range(k_sets)]
+            qkv = [rnd(N, (h + kv) * kd + kv * vd) for _ in range(k_sets)]
+            cs = ops.Rotary(rot, 1e6).table(ctx + N + 1, dev)
+            nb = N * 2 * 2 * ((h + kv) * kd + kv * vd)
+            report(group, f"Radivik, {name}", "rope_write",
+                   [lambda t=t, c=c: ops.rope_write(t, rows, c, cs, h, True, True, eps) for t, c in zip(qkv, caches)], nb)
+
+    # ------------------------------------------------------------------ norms and feed-forward
+    def row_case(N):
+        group = f"residual and norm, {N} rows"
+        w = torch.ones(W, device=dev, dtype=torch.bfloat16)
+        nb = N * W * 8
+        a = [(rnd(N, W), rnd(N, W)) for _ in range(sets(nb))]
+        report(group, "scaffold", "add_rms_norm", [lambda t=t: K.add_rms_norm(*t, w, 1e-6) for t in a], nb)
+        wf = torch.ones(W, device=dev)
+        nb = N * W * 12
+        a = [(rnd(N, W, dtype=torch.float32), rnd(N, W)) for _ in range(sets(nb))]
+        report(group, "Radivik", "scaled_add_norm", [lambda t=t: ops.scaled_add_norm(*t, wf, 2.0, 1e-6, torch.bfloat16) for t in a], nb)
+        for top in (2, 4):
+            idx = torch.randperm(N * top, generator=gen, device=dev).to(torch.int32).view(N, top)
+            nb = N * W * (10 + 2 * top)
+            a = [(rnd(N, W, dtype=torch.float32), rnd(N * top, W)) for _ in range(sets(nb))]
+            report(group, "Radivik", f"scaled_add_norm, sum of {top} experts",
+                   [lambda t=t: ops.scaled_add_norm(*t, wf, 2.0, 1e-6, torch.bfloat16, index=idx) for t in a], nb)
+
+    def mlp_case(N):
+        group = f"feed-forward, {N} rows"
+        k_sets = 4
+        xs = [rnd(N, W) for _ in range(k_sets)]
+        gu, dn = [rnd(2 * FF, W) for _ in range(k_sets)], [rnd(W, FF) for _ in range(k_sets)]
+        hs = [rnd(N, FF) for _ in range(k_sets)]
+        both = [rnd(N, 2 * FF) for _ in range(k_sets)]
+        report(group, "scaffold", "gate_up (cuBLAS)", [lambda i=i: K.linear(xs[i], gu[i]) for i in range(k_sets)],
+               2 * (2 * FF * W + N * W + 2 * N * FF), 2.0 * N * W * 2 * FF)
+        report(group, "scaffold", "silu_mul", [lambda i=i: K.silu_mul(both[i]) for i in range(k_sets)], 2 * 3 * N * FF)
+        report(group, "scaffold", "down (cuBLAS)", [lambda i=i: K.linear(hs[i], dn[i]) for i in range(k_sets)],
+               2 * (FF * W + N * FF + N * W), 2.0 * N * W * FF)
+        report(group, "scaffold", "whole", [lambda i=i: K.linear(K.silu_mul(K.linear(xs[i], gu[i])), dn[i]) for i in range(k_sets)],
+               2 * (3 * FF * W + 2 * N * W), 2.0 * N * W * 3 * FF)
+        del gu, dn, hs, both
+        for name, (*_, E, top, ff) in sizes.items():
+            x32 = [x.float() for x in xs]
+            exs = [ops.make_experts(rnd(E, W) * 0.05, rnd(E, ff, W), rnd(E, ff, W), rnd(E, W, ff), top, 7.0, GATE_SLOPE, torch.bfloat16, dev)
+                   for _ in range(2)]
+            total, tr = N * top, ops.expert_tile_rows(N, top, E, torch.bfloat16)
+            mt = ops.max_expert_tiles(total, E, tr)
+            ids, ranks, slots, scores = (torch.empty(total, dtype=torch.int32, device=dev) for _ in range(4))
+            tiles = torch.empty(1 + 3 * mt, dtype=torch.int32, device=dev)
+            lib = ops._lib_dec()
+            x_sorted, s_sorted = rnd(total, W), torch.empty(total, device=dev)
+            cnt = exs[0].counts
+
+            def route(i):
+                cnt.zero_()
+                lib.b200dec_router(x32[i].data_ptr(), exs[0].router.data_ptr(), N, W, E, top, ids.data_ptr(), scores.data_ptr(), ranks.data_ptr(),
+                                   cnt.data_ptr(), K._stream())
+
+            def spread(i):
+                lib.b200dec_dispatch(xs[i].data_ptr(), 2, ids.data_ptr(), scores.data_ptr(), ranks.data_ptr(), cnt.data_ptr(), N, W, E, top, tr,
+                                     x_sorted.data_ptr(), s_sorted.data_ptr(), slots.data_ptr(), tiles.data_ptr(), mt, K._stream())
+
+            who = f"Radivik, {name}"
+            report(group, who, "router (with a memset)", [lambda i=i: route(i) for i in range(k_sets)], N * W * 4 + E * W * 2, 0.0)
+            route(0)
+            report(group, who, "dispatch", [lambda i=i: spread(i) for i in range(k_sets)], N * W * 2 * (1 + top))
+            spread(0)
+            torch.cuda.synchronize()
+            used = int((cnt > 0).sum())
+            ha = rnd(total, ff)
+            report(group, who, "grouped gate_up + gated unit",
+                   [lambda e=e: ops.grouped_linear(x_sorted, e.gate_up, tiles, mt, tr, s_sorted, 7.0, GATE_SLOPE) for e in exs],
+                   2 * (used * 2 * ff * W + total * W + total * ff), 2.0 * total * W * 2 * ff)
+            report(group, who, "grouped down", [lambda e=e: ops.grouped_linear(ha, e.down, tiles, mt, tr) for e in exs],
+                   2 * (used * ff * W + total * ff + total * W), 2.0 * total * W * ff)
+
+            def whole(i, e):
+                e.counts.zero_()
+                ops.mixture(x32[i], xs[i], e)
+
+            report(group, who, "whole", [lambda i=i: whole(i, exs[i % 2]) for i in range(k_sets)],
+                   2 * (used * 3 * ff * W + 2 * N * W), 2.0 * total * W * 3 * ff)
+            del exs
+
+    # ------------------------------------------------------------------ whole steps
+    def model_case():
+        layers, vocab, prior, chunk, B, ctx = 8, 32768, 3072, 1024, 64, 4096
+        models = [("scaffold", model_class({"architecture": "DecoderScaffold"}).from_config(
+            {"hidden": W, "ffn": FF, "vocab": vocab, "layers": layers}, None, dev), PAGE)]
+        models += [(f"Radivik, {n}", model_class({"architecture": "Radivik"}).from_config(config(sz, layers, vocab), None, dev), page_r)
+                   for n, sz in sizes.items()]
+        for name, m, page in models:
+            P = ctx // page
+            caches = m.make_caches(B * P, page, ctx)
+            plan = S.plan_step([], [(prior, chunk)], chunk, 2)
+            table = torch.zeros(2, P, dtype=torch.int32)
+            table[0] = torch.arange(P)
+            inp = S.upload_step(plan, table, torch.randint(0, vocab, (chunk,)).tolist(), dev)
+            prefix = m.make_prefix(ctx)
+            prefix = None if prefix is None else S.PrefixScratch(*prefix, inp.cu_cached)
+            us = graph_us([lambda: m.step(caches, inp, inp.ids, inp.cached_lens, inp.block_table, inp.num_decoding, prefix)])
+            print(json.dumps({"case": f"prompt portion of {chunk} tokens on {prior}, {layers} layers", "model": name, "ms": round(us / 1e3, 3),
+                              "tokens_per_s": round(chunk / us * 1e6)}), flush=True)
+            tab = torch.randperm(B * P, generator=gen, device=dev).to(torch.int32).view(B, P)
+            ids, cached, nd = i32(list(range(B))), i32([ctx - 1] * B), i32([B])
+            us = graph_us([lambda: m.step(caches, None, ids, cached, tab, nd)])
+            print(json.dumps({"case": f"decode step of {B} entries of {ctx}, {layers} layers", "model": name, "ms": round(us / 1e3, 3),
+                              "tokens_per_s": round(B / us * 1e6), "status": K.check_status(dev)}), flush=True)
+            del caches
+
+    with ClockSampler(0) as clk:
+        for prior, chunk in ((3072, 992), (0, 992)):
+            prefill_case(prior, chunk)
+        for B, ctx in ((64, 4096), (8, 2048)):
+            decode_case(B, ctx)
+        write_case(64, True)
+        write_case(1024, False)
+        for N in (64, 1024, 4096):
+            row_case(N)
+        for N in (64, 1024, 4096):
+            mlp_case(N)
+        model_case()
+    print(json.dumps({"clocks": clk.summary(), "hbm_gbs": hbm / 1e9, "bf16_tflops": tf / 1e12, "data": "random weights and inputs"}), flush=True)
+
+
 def run_mixed(args):
     """--mixed: one chunked-prefill + decode step (seed 3) inside a random-init Qwen3-1.7B-shaped
     decoder (28 layers, hidden 2048, FFN 6144, vocab 151936, tied embeddings, weights ~N(0,0.02)):
@@ -1600,8 +1893,11 @@ def main():
     ap.add_argument("--dump", default=None, help="--phases: prefix of .npy files for the raw per-warp words")
     ap.add_argument("--linear", action="store_true", help="weight-streaming matmul for few rows beside cuBLAS")
     ap.add_argument("--phases", action="store_true", help="per-phase and per-SM times of the decode kernel (instrumented build)")
+    ap.add_argument("--radivik", action="store_true", help="the Radivik decoder beside the scaffold: kernels against their rooflines, whole steps")
     args = ap.parse_args()
-    if args.phases:
+    if args.radivik:
+        run_radivik(args)
+    elif args.phases:
         run_phases(args)
     elif args.linear:
         run_linear(args)

@@ -20,6 +20,16 @@ __device__ __forceinline__ void ld_elem4(const uint16_t* p, float (&f)[4]) {
   f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xFFFF0000u);
   f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xFFFF0000u);
 }
+// The same through L2 only.  With chained launches a kernel is brought up while the one before it still runs, so its
+// multiprocessor's L1 may hold a line that the predecessor read before another of its blocks wrote part of it.  Whatever the
+// predecessor produces next to (or over) what it reads is therefore loaded this way.
+__device__ __forceinline__ void ld_fresh4(const float* p, float (&f)[4]) {
+  const float4 v = __ldcg(reinterpret_cast<const float4*>(p));
+  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+__device__ __forceinline__ float ld_fresh(const float* p) { return __ldcg(p); }
+__device__ __forceinline__ int ld_fresh(const int32_t* p) { return __ldcg(p); }
+
 __device__ __forceinline__ void st_elem4(float* p, const float (&f)[4]) {
   *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
 }

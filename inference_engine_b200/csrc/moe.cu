@@ -6,29 +6,42 @@
 namespace b200kv {
 
 // ------------------------------------------------------------------ router
-// One block per kR rows, which it keeps in shared memory; a warp takes four experts at a time, its lanes run over the
-// channels, so a weight is read once per kR rows and a channel of x once per four experts.
+// One block per kR rows, which it keeps in shared memory.  A warp takes four experts at a time and, when there are fewer
+// groups of four than warps, a slice of the channels of them; its lanes run over the channels, so a weight is read once
+// per kR rows and a channel of x once per four experts.
 constexpr int kRtWarps = 8;
 constexpr int kRtExperts = 4;
 constexpr int kRtMaxExperts = 1024;
 
 template <int kR>
 __global__ void __launch_bounds__(kRtWarps * 32)
-router_kernel(const float* __restrict__ x, const uint16_t* __restrict__ w, int N, int width, int E, int top, int32_t* __restrict__ ids,
-              float* __restrict__ scores, int32_t* __restrict__ ranks, int32_t* __restrict__ counts) {
-  extern __shared__ float rt_smem[];
-  float* xs = rt_smem;               // [kR][width]
-  float* sc = xs + kR * width;       // [kR][E]
+router_kernel(const float* __restrict__ x, const uint16_t* __restrict__ w, int N, int width, int E, int top, int slices,
+              int32_t* __restrict__ ids, float* __restrict__ scores, int32_t* __restrict__ ranks, int32_t* __restrict__ counts) {
+  extern __shared__ __align__(16) float rt_smem[];
+  const int pitch = (width + 3) & ~3;
+  float* xs = rt_smem;                // [kR][pitch]
+  float* sc = xs + kR * pitch;        // [kR][E]
+  float* part = sc + kR * E;          // [slices][kR][E], only with slices > 1
   pdl_enter();
   pdl_wait();
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int r0 = blockIdx.x * kR, nr = min(kR, N - r0);
-  for (int i = tid; i < kR * width; i += kRtWarps * 32) {
-    const int r = i / width;
-    xs[i] = r < nr ? x[(long long)(r0 + r) * width + (i - r * width)] : 0.f;
+  for (int r = 0; r < kR; ++r) {
+    const float* src = x + (long long)(r0 + r) * width;
+    if (width % 4 == 0) {
+      for (int c = tid * 4; c < width; c += kRtWarps * 128) {
+        float f[4] = {0.f, 0.f, 0.f, 0.f};
+        if (r < nr) ld_fresh4(src + c, f);
+        st_elem4(xs + r * pitch + c, f);
+      }
+    } else {
+      for (int c = tid; c < width; c += kRtWarps * 32) xs[r * pitch + c] = r < nr ? ld_fresh(src + c) : 0.f;
+    }
   }
   __syncthreads();
-  for (int e0 = warp * kRtExperts; e0 < E; e0 += kRtWarps * kRtExperts) {
+  const int groups = (E + kRtExperts - 1) / kRtExperts;
+  for (int item = warp; item < groups * slices; item += kRtWarps) {
+    const int e0 = item / slices * kRtExperts, slice = item % slices;
     float acc[kRtExperts][kR];
 #pragma unroll
     for (int i = 0; i < kRtExperts; ++i)
@@ -37,35 +50,48 @@ router_kernel(const float* __restrict__ x, const uint16_t* __restrict__ w, int N
     const uint16_t* wp[kRtExperts];
 #pragma unroll
     for (int i = 0; i < kRtExperts; ++i) wp[i] = w + (long long)min(e0 + i, E - 1) * width;
-    if (width % 2 == 0) {
+    if (width % 4 == 0) {
+      const int per = (width / 4 + slices - 1) / slices * 4, hi = min(width, (slice + 1) * per);
 #pragma unroll 4
-      for (int c = 2 * lane; c < width; c += 64) {
-        float2 xv[kR];
+      for (int c = slice * per + 4 * lane; c < hi; c += 128) {
+        float wv[kRtExperts][4];
 #pragma unroll
-        for (int r = 0; r < kR; ++r) xv[r] = *reinterpret_cast<const float2*>(xs + r * width + c);
+        for (int i = 0; i < kRtExperts; ++i) ld_elem4(wp[i] + c, wv[i]);
 #pragma unroll
-        for (int i = 0; i < kRtExperts; ++i) {
-          const uint32_t u = *reinterpret_cast<const uint32_t*>(wp[i] + c);
-          const float lo = __uint_as_float(u << 16), hi = __uint_as_float(u & 0xFFFF0000u);
+        for (int r = 0; r < kR; ++r) {
+          float xv[4];
+          ld_elem4(xs + r * pitch + c, xv);
 #pragma unroll
-          for (int r = 0; r < kR; ++r) acc[i][r] = fmaf(hi, xv[r].y, fmaf(lo, xv[r].x, acc[i][r]));
+          for (int i = 0; i < kRtExperts; ++i)
+#pragma unroll
+            for (int k = 0; k < 4; ++k) acc[i][r] = fmaf(wv[i][k], xv[k], acc[i][r]);
         }
       }
     } else {
-      for (int c = lane; c < width; c += 32)
+      for (int c = slice * 32 + lane; c < width; c += 32 * slices)
 #pragma unroll
         for (int i = 0; i < kRtExperts; ++i)
 #pragma unroll
-          for (int r = 0; r < kR; ++r) acc[i][r] = fmaf(ld_elem(wp[i] + c), xs[r * width + c], acc[i][r]);
+          for (int r = 0; r < kR; ++r) acc[i][r] = fmaf(ld_elem(wp[i] + c), xs[r * pitch + c], acc[i][r]);
     }
+    float* dst = slices > 1 ? part + slice * kR * E : sc;
 #pragma unroll
     for (int i = 0; i < kRtExperts; ++i)
 #pragma unroll
       for (int r = 0; r < kR; ++r) {
         const float z = warp_sum(acc[i][r]);
-        // a score that is not a number (an idle row's left-overs) counts as the smallest one
-        if (lane == 0 && e0 + i < E) sc[r * E + e0 + i] = z == z ? 1.0f / (1.0f + expf(-z)) : 0.f;
+        if (lane == 0 && e0 + i < E) dst[r * E + e0 + i] = z;
       }
+  }
+  __syncthreads();
+  for (int i = tid; i < kR * E; i += kRtWarps * 32) {
+    float z = 0.f;
+    if (slices > 1)
+      for (int k = 0; k < slices; ++k) z += part[k * kR * E + i];
+    else
+      z = sc[i];
+    // a score that is not a number (an idle row's left-overs) counts as the smallest one
+    sc[i] = z == z ? 1.0f / (1.0f + expf(-z)) : 0.f;
   }
   __syncthreads();
   for (int r = warp; r < nr; r += kRtWarps) {
@@ -133,19 +159,22 @@ dispatch_kernel(const T* __restrict__ xb, const int32_t* __restrict__ ids, const
   const int tid = threadIdx.x;
   int base = 0, tbase = 0;
   for (int e0 = 0; e0 < E; e0 += kDpThreads) {
-    const int e = e0 + tid, n = e < E ? counts[e] : 0;
+    const int e = e0 + tid, n = e < E ? ld_fresh(counts + e) : 0;
     int sum;
     const int f = base + dp_scan(n, red, &sum);
     base += sum;
     if (e < E) first[e] = f;
     if (blockIdx.x == 0) {
-      const int nt = (n + tile_rows - 1) / tile_rows;
+      // an expert's run is cut evenly: a short last tile would cost almost as much as a full one
+      int nt = (n + tile_rows - 1) / tile_rows;
+      const int each = nt ? min(tile_rows, ((n + nt - 1) / nt + 15) / 16 * 16) : 1;
+      nt = (n + each - 1) / each;
       int t = tbase + dp_scan(nt, red, &sum);
       tbase += sum;
       for (int i = 0; i < nt && t < max_tiles; ++i, ++t) {
         tiles[1 + 3 * t] = e;
-        tiles[2 + 3 * t] = f + i * tile_rows;
-        tiles[3 + 3 * t] = min(tile_rows, n - i * tile_rows);
+        tiles[2 + 3 * t] = f + i * each;
+        tiles[3 + 3 * t] = min(each, n - i * each);
       }
     }
   }
@@ -156,7 +185,7 @@ dispatch_kernel(const T* __restrict__ xb, const int32_t* __restrict__ ids, const
     const T* src = xb + r * width;
     for (int j = 0; j < top; ++j) {
       const long long o = r * top + j;
-      const int place = first[ids[o]] + ranks[o];
+      const int place = first[ld_fresh(ids + o)] + ld_fresh(ranks + o);
       T* dst = x_sorted + (long long)place * width;
       if (width % kVec == 0) {
         for (int c = tid * kVec; c < width; c += kDpThreads * kVec) *reinterpret_cast<uint4*>(dst + c) = *reinterpret_cast<const uint4*>(src + c);
@@ -165,7 +194,7 @@ dispatch_kernel(const T* __restrict__ xb, const int32_t* __restrict__ ids, const
       }
       if (tid == 0) {
         slots[o] = place;
-        score_sorted[place] = scores[o];
+        score_sorted[place] = ld_fresh(scores + o);
       }
     }
   }
@@ -190,10 +219,10 @@ grouped_linear_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, con
   __shared__ float ws[kGsStep][kGsCols + 1];
   pdl_enter();
   pdl_wait();
-  const int num = tiles[0], tid = threadIdx.x, col = tid & 63, rg = tid >> 6;
+  const int num = ld_fresh(tiles), tid = threadIdx.x, col = tid & 63, rg = tid >> 6;
   const int o = blockIdx.x * kGsCols + col;
   for (int t = blockIdx.y; t < num; t += gridDim.y) {
-    const int e = tiles[1 + 3 * t], row0 = tiles[2 + 3 * t], nrows = tiles[3 + 3 * t];
+    const int e = ld_fresh(tiles + 1 + 3 * t), row0 = ld_fresh(tiles + 2 + 3 * t), nrows = ld_fresh(tiles + 3 + 3 * t);
     for (int sub = 0; sub < nrows; sub += kGsRows) {
       const int n = min(kGsRows, nrows - sub);
       float acc[8];
@@ -222,7 +251,7 @@ grouped_linear_simt_kernel(const T* __restrict__ x, const T* __restrict__ w, con
         const int rr = rg * 8 + i;
         const long long row = row0 + sub + rr;
         if (act) {  // neighbouring lanes hold gate (even output) and up (odd output)
-          const float s = rr < n ? score_sorted[row] : 0.f;
+          const float s = rr < n ? ld_fresh(score_sorted + row) : 0.f;
           const float mine = acc[i] * s, other = __shfl_xor_sync(0xffffffffu, mine, 1);
           if (rr < n && o < out_rows && (o & 1) == 0) st_elem(y + row * (out_rows / 2) + o / 2, gated_unit(mine, other, limit, slope));
         } else if (rr < n && o < out_rows) {
@@ -248,16 +277,19 @@ extern "C" int b200dec_router(const float* x, const void* router_w, int32_t num_
   if (num_rows < 0 || width < 1 || experts < 1 || experts > kRtMaxExperts || top < 1 || top > experts) return B200KV_E_SHAPE;
   if (!aligned(x, 16) || !aligned(router_w, 16)) return B200KV_E_ALIGN;
   cudaStream_t s = (cudaStream_t)stream;
-  const size_t smem8 = (size_t)8 * (width + experts) * 4, smem1 = (size_t)(width + experts) * 4;
+  const int groups = (experts + kRtExperts - 1) / kRtExperts;
+  const int slices = groups >= kRtWarps ? 1 : kRtWarps / groups;
+  const int extra = slices > 1 ? slices : 0;
+  const size_t smem1 = (size_t)((width + 3) / 4 * 4 + (1 + extra) * experts) * 4, smem8 = 8 * smem1;
   if (smem1 > 220 * 1024) return B200KV_E_RANGE;
   if (num_rows >= 1024 && smem8 <= 110 * 1024) {
     if (cudaFuncSetAttribute(router_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem8) != cudaSuccess) return B200KV_E_LAUNCH;
     return launch_result(launch_chained(router_kernel<8>, dim3((num_rows + 7) / 8), dim3(kRtWarps * 32), smem8, s, x, (const uint16_t*)router_w,
-                                        num_rows, width, experts, top, ids, scores, ranks, counts));
+                                        num_rows, width, experts, top, slices, ids, scores, ranks, counts));
   }
   if (cudaFuncSetAttribute(router_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1) != cudaSuccess) return B200KV_E_LAUNCH;
   return launch_result(launch_chained(router_kernel<1>, dim3(num_rows), dim3(kRtWarps * 32), smem1, s, x, (const uint16_t*)router_w, num_rows,
-                                      width, experts, top, ids, scores, ranks, counts));
+                                      width, experts, top, slices, ids, scores, ranks, counts));
 }
 
 extern "C" int b200dec_dispatch(const void* xb, int32_t elem, const int32_t* ids, const float* scores, const int32_t* ranks,

@@ -50,11 +50,29 @@ __device__ __forceinline__ void mg_mma(uint32_t d_tmem, uint64_t a_desc, uint64_
       ::"r"(d_tmem), "l"(a_desc), "l"(b_desc), "r"(idesc), "r"(acc) : "memory");
 }
 
+// Work item: a tile of one expert's rows and a block of its weight rows.  An entry of the list that does not fit (it would be
+// the product of an inconsistent routing) is reported and passed over, alike by every role.
+struct MgItem {
+  int e, row0, rows, m0;
+  bool ok;
+};
+template <int kN>
+__device__ __forceinline__ MgItem mg_item(const int32_t* tiles, int it, int blocks, int experts, int total_rows) {
+  const int t = it / blocks;
+  MgItem x;
+  x.m0 = (it - t * blocks) * kMgM;
+  x.e = ld_fresh(tiles + 1 + 3 * t);
+  x.row0 = ld_fresh(tiles + 2 + 3 * t);
+  x.rows = ld_fresh(tiles + 3 + 3 * t);
+  x.ok = x.e >= 0 && x.e < experts && x.rows >= 1 && x.rows <= kN && x.row0 >= 0 && x.row0 <= total_rows - x.rows;
+  return x;
+}
+
 template <int kN, bool kAct>
 __global__ void __launch_bounds__(kMgThreads, 1)
 grouped_linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid_constant__ CUtensorMap tm_x, const int32_t* __restrict__ tiles,
-                          int out_rows, int steps, const float* __restrict__ score_sorted, float limit, float slope,
-                          uint16_t* __restrict__ y, int32_t* status) {
+                          int max_tiles, int experts, int total_rows, int out_rows, int steps, const float* __restrict__ score_sorted,
+                          float limit, float slope, uint16_t* __restrict__ y, int32_t* status) {
   using S = MgShape<kN>;
   extern __shared__ uint8_t mg_raw[];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -87,23 +105,27 @@ grouped_linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid
   asm volatile("ld.shared.u32 %0, [%1];\n" : "=r"(tmem) : "r"(slot_word) : "memory");
   pdl_wait();  // the tile list and the rows come from the kernels before this one
   const int blocks = (out_rows + kMgM - 1) / kMgM;
-  const int items = tiles[0] * blocks;
+  const int items = min(max(ld_fresh(tiles), 0), max_tiles) * blocks;
 
   if (warp == 0) {
     if (lane == 0) {
       int i = 0;
       bool live = true;
       for (int it = blockIdx.x; it < items && live; it += gridDim.x) {
-        const int t = it / blocks, m0 = (it - t * blocks) * kMgM;
-        const int e = tiles[1 + 3 * t], row0 = tiles[2 + 3 * t], boxes = (tiles[3 + 3 * t] + S::kBox - 1) / S::kBox;
+        const MgItem x = mg_item<kN>(tiles, it, blocks, experts, total_rows);
+        if (!x.ok) {
+          if (status) atomicOr(status, B200KV_S_BAD_POSITION);
+          continue;
+        }
+        const int boxes = (x.rows + S::kBox - 1) / S::kBox;
         const uint32_t bytes = kMgWBytes + (uint32_t)boxes * S::kBox * 128;
         for (int k = 0; k < steps; ++k, ++i) {
           const int s = i % S::kStages;
           if (i >= S::kStages && !dt_mbar_wait(bar_empty(s), (i / S::kStages - 1) & 1)) { live = false; break; }
           const uint32_t dst = base + s * S::kSlot;
           dt_expect_tx(bar_full(s), bytes);
-          dt_tma_2d(dst, &tm_w, k * kMgStep, e * out_rows + m0, bar_full(s));
-          for (int b = 0; b < boxes; ++b) dt_tma_2d(dst + kMgWBytes + b * S::kBox * 128, &tm_x, k * kMgStep, row0 + b * S::kBox, bar_full(s));
+          dt_tma_2d(dst, &tm_w, k * kMgStep, x.e * out_rows + x.m0, bar_full(s));
+          for (int b = 0; b < boxes; ++b) dt_tma_2d(dst + kMgWBytes + b * S::kBox * 128, &tm_x, k * kMgStep, x.row0 + b * S::kBox, bar_full(s));
         }
       }
       pdl_trigger();  // nothing left to fetch: the next kernel may be brought up
@@ -116,9 +138,11 @@ grouped_linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid
     if (lane == 0) {
       int i = 0, n = 0;
       bool live = true;
-      for (int it = blockIdx.x; it < items && live; it += gridDim.x, ++n) {
+      for (int it = blockIdx.x; it < items && live; it += gridDim.x) {
+        const MgItem x = mg_item<kN>(tiles, it, blocks, experts, total_rows);
+        if (!x.ok) continue;
         const int buf = n & 1;
-        const uint32_t idesc = mg_idesc((uint32_t)((tiles[3 + 3 * (it / blocks)] + 15) & ~15));
+        const uint32_t idesc = mg_idesc((uint32_t)((x.rows + 15) & ~15));
         if (n >= 2 && !dt_mbar_wait(bar_free(buf), (n / 2 - 1) & 1)) break;
         asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
         for (int k = 0; k < steps; ++k, ++i) {
@@ -132,15 +156,17 @@ grouped_linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid
           mg_commit(bar_empty(s));
         }
         if (live) mg_commit(bar_done(buf));
+        ++n;
       }
     }
   } else {
     int n = 0;
     const int wl = warp & 3;  // tensor-memory lanes 32 wl ..
-    for (int it = blockIdx.x; it < items; it += gridDim.x, ++n) {
-      const int buf = n & 1, t = it / blocks;
-      const int o = (it - t * blocks) * kMgM + 32 * wl + lane;  // this lane's weight row
-      const int row0 = tiles[2 + 3 * t], rows = tiles[3 + 3 * t];
+    for (int it = blockIdx.x; it < items; it += gridDim.x) {
+      const MgItem x = mg_item<kN>(tiles, it, blocks, experts, total_rows);
+      if (!x.ok) continue;
+      const int buf = n & 1, row0 = x.row0, rows = x.rows;
+      const int o = x.m0 + 32 * wl + lane;  // this lane's weight row
       const bool ok = dt_mbar_wait(bar_done(buf), (n / 2) & 1);
       if (!__all_sync(0xffffffffu, ok)) {
         if (lane == 0 && status) atomicOr(status, B200KV_S_TIMEOUT);
@@ -151,7 +177,7 @@ grouped_linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid
         uint32_t u[32];
         t5_ld32(tmem + buf * kN + c0 + ((uint32_t)(32 * wl) << 16), u);
         if (kAct) {
-          const float sl = c0 + lane < rows ? score_sorted[row0 + c0 + lane] : 0.f;
+          const float sl = c0 + lane < rows ? ld_fresh(score_sorted + row0 + c0 + lane) : 0.f;
           const bool odd = lane & 1;
           uint16_t* dst = y + (long long)(row0 + c0 + odd) * (out_rows / 2) + o / 2;
 #pragma unroll
@@ -176,6 +202,7 @@ grouped_linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid
       asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
       __syncwarp();
       if (lane == 0) dt_mbar_arrive(bar_free(buf));
+      ++n;
     }
   }
   asm volatile("tcgen05.fence::before_thread_sync;\n" ::: "memory");
@@ -184,21 +211,21 @@ grouped_linear_tc5_kernel(const __grid_constant__ CUtensorMap tm_w, const __grid
 }
 
 template <int kN, bool kAct>
-static int mg_launch(const CUtensorMap& tm_w, const CUtensorMap& tm_x, const int32_t* tiles, int grid, int out_rows, int steps,
+static int mg_launch(const CUtensorMap& tm_w, const CUtensorMap& tm_x, const int32_t* tiles, int grid, int max_tiles, int experts, int total_rows, int out_rows, int steps,
                      const float* score_sorted, float limit, float slope, void* y, int32_t* status, cudaStream_t stream) {
   if (cudaFuncSetAttribute(grouped_linear_tc5_kernel<kN, kAct>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)MgShape<kN>::kSmem) !=
       cudaSuccess)
     return B200KV_E_LAUNCH;
   return launch_result(launch_chained(grouped_linear_tc5_kernel<kN, kAct>, dim3(grid), dim3(kMgThreads), MgShape<kN>::kSmem, stream, tm_w, tm_x,
-                                      tiles, out_rows, steps, score_sorted, limit, slope, (uint16_t*)y, status));
+                                      tiles, max_tiles, experts, total_rows, out_rows, steps, score_sorted, limit, slope, (uint16_t*)y, status));
 }
 
 int launch_grouped_linear_tc5(const void* x, const void* w, const int32_t* tiles, int max_tiles, int tile_rows, int total_rows, int experts,
                               int out_rows, int width, const float* score_sorted, int act, float limit, float slope, void* y, int sms,
                               int32_t* status, cudaStream_t stream) {
-  if (tile_rows != 64 && tile_rows != 256) return B200KV_E_SHAPE;
+  if (tile_rows > 256) return B200KV_E_SHAPE;
   if ((long long)experts * out_rows > 0x7FFFFFFFll) return B200KV_E_RANGE;
-  const int box = tile_rows == 256 ? MgShape<256>::kBox : MgShape<64>::kBox;
+  const int box = tile_rows > 64 ? MgShape<256>::kBox : MgShape<64>::kBox;
   CUtensorMap tm_w, tm_x;
   const uint64_t wd[2] = {(uint64_t)width, (uint64_t)experts * out_rows}, xd[2] = {(uint64_t)width, (uint64_t)total_rows};
   const uint64_t st[1] = {(uint64_t)width};
@@ -206,11 +233,11 @@ int launch_grouped_linear_tc5(const void* x, const void* w, const int32_t* tiles
   if (!dt_make_map(&tm_w, w, 2, wd, st, wb) || !dt_make_map(&tm_x, x, 2, xd, st, xb)) return B200KV_E_LAUNCH;
   const long long items = (long long)max_tiles * ((out_rows + kMgM - 1) / kMgM);
   const int grid = (int)(items < sms ? items : sms), steps = (width + kMgStep - 1) / kMgStep;
-  if (tile_rows == 256)
-    return act ? mg_launch<256, true>(tm_w, tm_x, tiles, grid, out_rows, steps, score_sorted, limit, slope, y, status, stream)
-               : mg_launch<256, false>(tm_w, tm_x, tiles, grid, out_rows, steps, score_sorted, limit, slope, y, status, stream);
-  return act ? mg_launch<64, true>(tm_w, tm_x, tiles, grid, out_rows, steps, score_sorted, limit, slope, y, status, stream)
-             : mg_launch<64, false>(tm_w, tm_x, tiles, grid, out_rows, steps, score_sorted, limit, slope, y, status, stream);
+  if (tile_rows > 64)
+    return act ? mg_launch<256, true>(tm_w, tm_x, tiles, grid, max_tiles, experts, total_rows, out_rows, steps, score_sorted, limit, slope, y, status, stream)
+               : mg_launch<256, false>(tm_w, tm_x, tiles, grid, max_tiles, experts, total_rows, out_rows, steps, score_sorted, limit, slope, y, status, stream);
+  return act ? mg_launch<64, true>(tm_w, tm_x, tiles, grid, max_tiles, experts, total_rows, out_rows, steps, score_sorted, limit, slope, y, status, stream)
+             : mg_launch<64, false>(tm_w, tm_x, tiles, grid, max_tiles, experts, total_rows, out_rows, steps, score_sorted, limit, slope, y, status, stream);
 }
 
 }  // namespace b200kv

@@ -7,17 +7,23 @@ namespace b200kv {
 constexpr int kRwWarps = 8;
 constexpr int kRwMaxPairs = 16;  // a lane holds up to 32 channels: heads of up to 1024
 
+__device__ __forceinline__ float2 rw_load2(const uint16_t* p) {
+  const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
+  return make_float2(__uint_as_float(u << 16), __uint_as_float(u & 0xFFFF0000u));
+}
+__device__ __forceinline__ float2 rw_load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
+
 // One warp per (row, head), heads in the order q | k | v.  A lane owns channels 2 * lane + 64 * i and the next one.
-template <typename T>
+// kPairs: head sizes, half and the row stride are even, so both channels are loaded and rotated together.
+template <typename T, bool kPairs>
 __global__ void __launch_bounds__(kRwWarps * 32)
 rope_write_kernel(const T* __restrict__ qkv, long long qkv_stride, b200dec_rows rows, DecCache c, const float* __restrict__ cos_sin,
                   int table_len, int half, int heads, int write_kv, int unit_norm, float eps, T* __restrict__ q_out, int32_t* status) {
   pdl_enter();
   const int hkv = write_kv ? c.heads : 0, per_row = heads + 2 * hkv;
-  const long long item = (long long)blockIdx.x * kRwWarps + (threadIdx.x >> 5);
-  const int lane = threadIdx.x & 31;
-  if (item >= (long long)rows.num_rows * per_row) return;
-  const int r = (int)(item / per_row), j = (int)(item - (long long)r * per_row);
+  const int item = blockIdx.x * kRwWarps + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (item >= rows.num_rows * per_row) return;
+  const int r = item / per_row, j = item - r * per_row;
   const int kind = j < heads ? 0 : (j < heads + hkv ? 1 : 2);  // q, k, v
   int seq = r, pos;
   if (rows.seq_ids) {
@@ -65,7 +71,23 @@ rope_write_kernel(const T* __restrict__ qkv, long long qkv_stride, b200dec_rows 
   const float2* cs = reinterpret_cast<const float2*>(cos_sin) + (long long)pos * half;
 #pragma unroll
   for (int i = 0; i < kRwMaxPairs; ++i) {
-    if (64 * i < dim) {
+    y[i][0] = y[i][1] = 0.f;
+    if (kPairs && 64 * i < dim) {
+      const int ch = 64 * i + 2 * lane;
+      if (ch < dim) {
+        float2 v = rw_load2(src + ch);
+        if (kind < 2 && ch < 2 * half) {
+          const bool low = ch < half;
+          const float2 other = rw_load2(src + (low ? ch + half : ch - half));
+          const float4 a = *reinterpret_cast<const float4*>(cs + (low ? ch : ch - half));  // cos, sin of both
+          const float s0 = low ? -a.y : a.y, s1 = low ? -a.w : a.w;
+          v = make_float2(v.x * a.x + other.x * s0, v.y * a.z + other.y * s1);
+        }
+        y[i][0] = v.x;
+        y[i][1] = v.y;
+        ss = fmaf(v.x, v.x, fmaf(v.y, v.y, ss));
+      }
+    } else if (64 * i < dim) {
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int ch = 64 * i + 2 * lane + e;
@@ -215,16 +237,18 @@ extern "C" int b200dec_rope_write(const void* qkv, int64_t qkv_stride, const b20
   if (!aligned(q_out, 16) || !aligned(cos_sin, 8)) return B200KV_E_ALIGN;
   const long long items = (long long)rows->num_rows * (heads + (write_kv ? 2 * cache->kv_heads : 0));
   const long long blocks = (items + kRwWarps - 1) / kRwWarps;
-  if (blocks > 0x7FFFFFFFll) return B200KV_E_RANGE;
+  if (items > 0x7FFFFFF0ll) return B200KV_E_RANGE;
   const DecCache c = dec_view(cache, table);
   cudaStream_t s = (cudaStream_t)stream;
+  const bool pairs = cache->k_dim % 2 == 0 && cache->v_dim % 2 == 0 && half % 2 == 0 && qkv_stride % 2 == 0 &&
+                     aligned(qkv, 2 * cache->elem) && aligned(cos_sin, 16);
+  auto run = [&](auto* kernel, auto* in, auto* q) {
+    return launch_result(launch_chained(kernel, dim3((unsigned)blocks), dim3(kRwWarps * 32), 0, s, in, (long long)qkv_stride, *rows, c, cos_sin,
+                                        table_len, half, heads, write_kv, unit_norm, eps, q, status));
+  };
   if (cache->elem == 2)
-    return launch_result(launch_chained(rope_write_kernel<uint16_t>, dim3((unsigned)blocks), dim3(kRwWarps * 32), 0, s, (const uint16_t*)qkv,
-                                        (long long)qkv_stride, *rows, c, cos_sin, table_len, half, heads, write_kv, unit_norm, eps,
-                                        (uint16_t*)q_out, status));
-  return launch_result(launch_chained(rope_write_kernel<float>, dim3((unsigned)blocks), dim3(kRwWarps * 32), 0, s, (const float*)qkv,
-                                      (long long)qkv_stride, *rows, c, cos_sin, table_len, half, heads, write_kv, unit_norm, eps,
-                                      (float*)q_out, status));
+    return run(pairs ? rope_write_kernel<uint16_t, true> : rope_write_kernel<uint16_t, false>, (const uint16_t*)qkv, (uint16_t*)q_out);
+  return run(pairs ? rope_write_kernel<float, true> : rope_write_kernel<float, false>, (const float*)qkv, (float*)q_out);
 }
 
 extern "C" int b200dec_attn_rows(const void* q, const b200dec_cache* cache, const b200kv_table* table, const b200dec_rows* rows,

@@ -6,7 +6,7 @@
 namespace b200kv {
 
 constexpr int kRowThreads = 256;
-constexpr int kRowChunks = 8;  // the register path holds rows of up to 256 * 4 * 8 = 8192 channels
+constexpr int kRowChunks = 8;  // the register path holds rows of up to 256 * 4 * 8 = 8192 channels (2 chunks: 2048)
 
 __device__ __forceinline__ float row_sum(float v) {
   __shared__ float part[kRowThreads / 32];
@@ -49,28 +49,28 @@ embed_kernel(const T* __restrict__ table, const int32_t* __restrict__ ids, float
 }
 
 // The registers path: width % 4 == 0 and width <= 8192.
-template <typename T>
+template <typename T, int kChunks>
 __global__ void __launch_bounds__(kRowThreads)
-scaled_add_norm_kernel(const float* __restrict__ x, const T* __restrict__ delta, const int32_t* __restrict__ index, int top,
-                       const float* __restrict__ weight, float alpha, float eps, float* __restrict__ x_out, T* __restrict__ xb_out,
+scaled_add_norm_kernel(const float* x, const T* __restrict__ delta, const int32_t* __restrict__ index, int top,
+                       const float* __restrict__ weight, float alpha, float eps, float* x_out, T* __restrict__ xb_out,
                        int width, int32_t* __restrict__ zero, int num_zero) {
   pdl_enter();
   pdl_wait();
   const long long r = blockIdx.x;
   if (zero && blockIdx.x == 0)
     for (int i = threadIdx.x; i < num_zero; i += kRowThreads) zero[i] = 0;
-  float s[kRowChunks][4];
+  float s[kChunks][4];
   float ss = 0.f;
 #pragma unroll
-  for (int c = 0; c < kRowChunks; ++c) {
+  for (int c = 0; c < kChunks; ++c) {
     const int col = (c * kRowThreads + threadIdx.x) * 4;
     if (col < width) {
-      ld_elem4(x + r * width + col, s[c]);
+      ld_fresh4(x + r * width + col, s[c]);
 #pragma unroll
       for (int i = 0; i < 4; ++i) s[c][i] *= alpha;
       if (delta) {
         for (int j = 0; j < top; ++j) {
-          const long long row = index ? index[r * top + j] : r;
+          const long long row = index ? ld_fresh(index + r * top + j) : r;
           float d[4];
           ld_elem4(delta + row * width + col, d);
 #pragma unroll
@@ -83,7 +83,7 @@ scaled_add_norm_kernel(const float* __restrict__ x, const T* __restrict__ delta,
   }
   const float inv = 1.0f / sqrtf(row_sum(ss) / (float)width + eps);
 #pragma unroll
-  for (int c = 0; c < kRowChunks; ++c) {
+  for (int c = 0; c < kChunks; ++c) {
     const int col = (c * kRowThreads + threadIdx.x) * 4;
     if (col < width) {
       float w[4];
@@ -99,8 +99,8 @@ scaled_add_norm_kernel(const float* __restrict__ x, const T* __restrict__ delta,
 // Any width: the sums are kept in dynamic shared memory.
 template <typename T>
 __global__ void __launch_bounds__(kRowThreads)
-scaled_add_norm_any_kernel(const float* __restrict__ x, const T* __restrict__ delta, const int32_t* __restrict__ index, int top,
-                           const float* __restrict__ weight, float alpha, float eps, float* __restrict__ x_out,
+scaled_add_norm_any_kernel(const float* x, const T* __restrict__ delta, const int32_t* __restrict__ index, int top,
+                           const float* __restrict__ weight, float alpha, float eps, float* x_out,
                            T* __restrict__ xb_out, int width, int32_t* __restrict__ zero, int num_zero) {
   extern __shared__ float srow[];
   pdl_enter();
@@ -110,9 +110,9 @@ scaled_add_norm_any_kernel(const float* __restrict__ x, const T* __restrict__ de
     for (int i = threadIdx.x; i < num_zero; i += kRowThreads) zero[i] = 0;
   float ss = 0.f;
   for (int c = threadIdx.x; c < width; c += kRowThreads) {
-    float s = alpha * x[r * width + c];
+    float s = alpha * ld_fresh(x + r * width + c);
     if (delta)
-      for (int j = 0; j < top; ++j) s += ld_elem(delta + (index ? (long long)index[r * top + j] : r) * width + c);
+      for (int j = 0; j < top; ++j) s += ld_elem(delta + (index ? (long long)ld_fresh(index + r * top + j) : r) * width + c);
     srow[c] = s;
     ss = fmaf(s, s, ss);
   }
@@ -128,8 +128,11 @@ template <typename T>
 static int run_scaled_add_norm(const float* x, const void* delta, const int32_t* index, int top, const float* weight, float alpha,
                                float eps, float* x_out, void* xb_out, int rows, int width, int32_t* zero, int num_zero,
                                cudaStream_t stream) {
+  if (width % 4 == 0 && width <= kRowThreads * 4 * 2)
+    return launch_result(launch_chained(scaled_add_norm_kernel<T, 2>, dim3(rows), dim3(kRowThreads), 0, stream, x, (const T*)delta, index,
+                                        top, weight, alpha, eps, x_out, (T*)xb_out, width, zero, num_zero));
   if (width % 4 == 0 && width <= kRowThreads * 4 * kRowChunks)
-    return launch_result(launch_chained(scaled_add_norm_kernel<T>, dim3(rows), dim3(kRowThreads), 0, stream, x, (const T*)delta, index,
+    return launch_result(launch_chained(scaled_add_norm_kernel<T, kRowChunks>, dim3(rows), dim3(kRowThreads), 0, stream, x, (const T*)delta, index,
                                         top, weight, alpha, eps, x_out, (T*)xb_out, width, zero, num_zero));
   const size_t smem = (size_t)width * 4;
   if (smem > 200 * 1024) return B200KV_E_RANGE;

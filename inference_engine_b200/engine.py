@@ -293,7 +293,6 @@ class Engine:
             r.cached_len += len(toks)
         with self.torch.inference_mode():
             if not rows:
-                self.torch.cuda.synchronize()
                 return self.torch.empty(0, self.model.vocab)
             return self.model.logits(out.hidden[self.torch.tensor(rows, device=self.device)]).float().cpu()
 

@@ -267,12 +267,20 @@ def make_experts(router, gates, ups, downs, top: int, limit: float, slope: float
                    torch.zeros(E, dtype=torch.int32, device=device))
 
 
-def expert_tile_rows(num_rows: int, top: int, dtype) -> int:
-    """Rows of an expert's tile: 256 for prompt-sized steps (the widest tcgen05 tile), 64 for small ones, where weights
-    are streamed and a narrow tile leaves shared memory for a deeper ring."""
+def expert_tile_rows(num_rows: int, top: int, experts: int, dtype) -> int:
+    """Most rows of an expert's tile: up to 256 for prompt-sized steps (the widest tcgen05 tile; 128 when that leaves few
+    tiles to spread over the GPU), 64 for small ones, where weights are streamed and a narrow tile leaves shared memory
+    for a deeper ring."""
     if dtype == torch.float32:
         return 32
-    return 64 if num_rows * top <= 512 else 256
+    total = num_rows * top
+    if total <= 512 or total <= 48 * experts:
+        return 64
+    return 128 if total <= 4096 else 256
+
+
+def max_expert_tiles(total: int, experts: int, tile_rows: int) -> int:
+    return total // tile_rows + min(experts, total)
 
 
 def grouped_linear(x, w, tiles, max_tiles, tile_rows, scores=None, limit=0.0, slope=0.0, variant: int | None = None):
@@ -301,10 +309,11 @@ def mixture(x: torch.Tensor, xb: torch.Tensor, ex: Experts, variant: int | None 
     lib, dev = _lib_dec(), x.device
     N, W = x.shape
     total, E = N * ex.top, ex.num
-    tile_rows = expert_tile_rows(N, ex.top, xb.dtype)
-    max_tiles = total // tile_rows + min(E, total)
-    meta = torch.empty(4 * total + 1 + 3 * max_tiles, dtype=torch.int32, device=dev)
-    ids, ranks, slots, scores, tiles = meta.split([total, total, total, total, 1 + 3 * max_tiles])
+    tile_rows = expert_tile_rows(N, ex.top, E, xb.dtype)
+    max_tiles = max_expert_tiles(total, E, tile_rows)
+    # separate allocations: no kernel of the chain reads a cache line that the next one's input shares
+    ids, ranks, slots, scores = (torch.empty(total, dtype=torch.int32, device=dev) for _ in range(4))
+    tiles = torch.empty(1 + 3 * max_tiles, dtype=torch.int32, device=dev)
     score_sorted = torch.empty(total, dtype=torch.float32, device=dev)
     rc = lib.b200dec_router(x.data_ptr(), ex.router.data_ptr(), N, W, E, ex.top, ids.data_ptr(), scores.data_ptr(), ranks.data_ptr(),
                             ex.counts.data_ptr(), K._stream())

@@ -198,3 +198,24 @@ def test_command_line_and_trace_replay(tmp_path):
     for n, at in ((0, [0, 8]), (2, [11]), (3, [20])):
         got = np.fromfile(res / f"{n}.f32", "<f4").reshape(len(at), cfg["vocab"])
         assert H.error(got, want[at]).max() < H.TOLERANCE[torch.float32]
+
+
+def test_chained_launches_change_nothing():
+    """Kernels brought up while their predecessor runs: the same bits, prompts and decoding, with and without."""
+    from inference_engine_b200 import kernels as K
+
+    for cfg in (CONFIGS["one_expert"], CONFIGS["many_heads"], H.config([H.layer(experts=16, top=3, ff=72)] * 3, width=192)):
+        w = H.weights(cfg, 11)
+        m = H.model(cfg, w, torch.bfloat16)
+        tokens = prompt(420, cfg["vocab"], 5)
+        outs = []
+        try:
+            for chained in (False, True, True):
+                K.set_early_start(chained)
+                junk = torch.full((1 << 22,), -1, dtype=torch.int32, device="cuda")  # scratch memory starts as nonsense
+                del junk
+                outs.append(H.feed(H.engine(m), tokens, [380] + list(range(381, 420))))
+        finally:
+            K.set_early_start(False)
+        assert np.array_equal(outs[0], outs[1]) and np.array_equal(outs[0], outs[2])
+        H.status_clear()
