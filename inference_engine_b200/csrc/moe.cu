@@ -14,7 +14,7 @@ constexpr int kRtExperts = 4;
 constexpr int kRtMaxExperts = 1024;
 
 template <int kR>
-__global__ void __launch_bounds__(kRtWarps * 32)
+__global__ void __launch_bounds__(kRtWarps * 32, 4)
 router_kernel(const float* __restrict__ x, const uint16_t* __restrict__ w, int N, int width, int E, int top, int slices,
               int32_t* __restrict__ ids, float* __restrict__ scores, int32_t* __restrict__ ranks, int32_t* __restrict__ counts) {
   extern __shared__ __align__(16) float rt_smem[];
@@ -52,7 +52,7 @@ router_kernel(const float* __restrict__ x, const uint16_t* __restrict__ w, int N
     for (int i = 0; i < kRtExperts; ++i) wp[i] = w + (long long)min(e0 + i, E - 1) * width;
     if (width % 4 == 0) {
       const int per = (width / 4 + slices - 1) / slices * 4, hi = min(width, (slice + 1) * per);
-#pragma unroll 4
+#pragma unroll 2
       for (int c = slice * per + 4 * lane; c < hi; c += 128) {
         float wv[kRtExperts][4];
 #pragma unroll
@@ -280,11 +280,11 @@ extern "C" int b200dec_router(const float* x, const void* router_w, int32_t num_
   const int groups = (experts + kRtExperts - 1) / kRtExperts;
   const int slices = groups >= kRtWarps ? 1 : kRtWarps / groups;
   const int extra = slices > 1 ? slices : 0;
-  const size_t smem1 = (size_t)((width + 3) / 4 * 4 + (1 + extra) * experts) * 4, smem8 = 8 * smem1;
+  const size_t smem1 = (size_t)((width + 3) / 4 * 4 + (1 + extra) * experts) * 4, smem4 = 4 * smem1;
   if (smem1 > 220 * 1024) return B200KV_E_RANGE;
-  if (num_rows >= 1024 && smem8 <= 110 * 1024) {
-    if (cudaFuncSetAttribute(router_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem8) != cudaSuccess) return B200KV_E_LAUNCH;
-    return launch_result(launch_chained(router_kernel<8>, dim3((num_rows + 7) / 8), dim3(kRtWarps * 32), smem8, s, x, (const uint16_t*)router_w,
+  if (num_rows >= 512 && smem4 <= 72 * 1024) {
+    if (cudaFuncSetAttribute(router_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem4) != cudaSuccess) return B200KV_E_LAUNCH;
+    return launch_result(launch_chained(router_kernel<4>, dim3((num_rows + 3) / 4), dim3(kRtWarps * 32), smem4, s, x, (const uint16_t*)router_w,
                                         num_rows, width, experts, top, slices, ids, scores, ranks, counts));
   }
   if (cudaFuncSetAttribute(router_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1) != cudaSuccess) return B200KV_E_LAUNCH;

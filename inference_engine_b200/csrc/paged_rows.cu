@@ -5,7 +5,7 @@
 namespace b200kv {
 
 constexpr int kRwWarps = 8;
-constexpr int kRwMaxPairs = 16;  // a lane holds up to 32 channels: heads of up to 1024
+constexpr int kRwMaxPairs = 16;  // a lane holds up to 32 channels: heads of up to 1024 (2: heads of up to 128)
 
 __device__ __forceinline__ float2 rw_load2(const uint16_t* p) {
   const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
@@ -15,7 +15,7 @@ __device__ __forceinline__ float2 rw_load2(const float* p) { return *reinterpret
 
 // One warp per (row, head), heads in the order q | k | v.  A lane owns channels 2 * lane + 64 * i and the next one.
 // kPairs: head sizes, half and the row stride are even, so both channels are loaded and rotated together.
-template <typename T, bool kPairs>
+template <typename T, bool kPairs, int kMax>
 __global__ void __launch_bounds__(kRwWarps * 32)
 rope_write_kernel(const T* __restrict__ qkv, long long qkv_stride, b200dec_rows rows, DecCache c, const float* __restrict__ cos_sin,
                   int table_len, int half, int heads, int write_kv, int unit_norm, float eps, T* __restrict__ q_out, int32_t* status) {
@@ -66,11 +66,11 @@ rope_write_kernel(const T* __restrict__ qkv, long long qkv_stride, b200dec_rows 
   }
   pdl_wait();
   const T* src = qkv + r * qkv_stride + src_off;
-  float y[kRwMaxPairs][2];
+  float y[kMax][2];
   float ss = 0.f;
   const float2* cs = reinterpret_cast<const float2*>(cos_sin) + (long long)pos * half;
 #pragma unroll
-  for (int i = 0; i < kRwMaxPairs; ++i) {
+  for (int i = 0; i < kMax; ++i) {
     y[i][0] = y[i][1] = 0.f;
     if (kPairs && 64 * i < dim) {
       const int ch = 64 * i + 2 * lane;
@@ -109,7 +109,7 @@ rope_write_kernel(const T* __restrict__ qkv, long long qkv_stride, b200dec_rows 
   float inv = 1.f;
   if (kind < 2 && unit_norm) inv = 1.0f / sqrtf(warp_sum(ss) / (float)dim + eps);
 #pragma unroll
-  for (int i = 0; i < kRwMaxPairs; ++i) {
+  for (int i = 0; i < kMax; ++i) {
     const int ch = 64 * i + 2 * lane;
     if (ch < row_len) {  // row_len is even; channels behind dim are zero
       if (sizeof(T) == 2)
@@ -246,9 +246,12 @@ extern "C" int b200dec_rope_write(const void* qkv, int64_t qkv_stride, const b20
     return launch_result(launch_chained(kernel, dim3((unsigned)blocks), dim3(kRwWarps * 32), 0, s, in, (long long)qkv_stride, *rows, c, cos_sin,
                                         table_len, half, heads, write_kv, unit_norm, eps, q, status));
   };
-  if (cache->elem == 2)
-    return run(pairs ? rope_write_kernel<uint16_t, true> : rope_write_kernel<uint16_t, false>, (const uint16_t*)qkv, (uint16_t*)q_out);
-  return run(pairs ? rope_write_kernel<float, true> : rope_write_kernel<float, false>, (const float*)qkv, (float*)q_out);
+  if (cache->elem == 2) {
+    if (pairs && cache->k_row <= 128 && cache->v_row <= 128) return run(rope_write_kernel<uint16_t, true, 2>, (const uint16_t*)qkv, (uint16_t*)q_out);
+    return run(pairs ? rope_write_kernel<uint16_t, true, kRwMaxPairs> : rope_write_kernel<uint16_t, false, kRwMaxPairs>, (const uint16_t*)qkv,
+               (uint16_t*)q_out);
+  }
+  return run(pairs ? rope_write_kernel<float, true, kRwMaxPairs> : rope_write_kernel<float, false, kRwMaxPairs>, (const float*)qkv, (float*)q_out);
 }
 
 extern "C" int b200dec_attn_rows(const void* q, const b200dec_cache* cache, const b200kv_table* table, const b200dec_rows* rows,

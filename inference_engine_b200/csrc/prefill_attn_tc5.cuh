@@ -289,6 +289,7 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
     const uint16_t* kown = k + (long long)seq_start * k_sn + hk * k_sh;
     const uint16_t* vown = v + (long long)seq_start * v_sn + hk * v_sh;
     bool live = true;
+    int win_base = -1, win_id = 0;  // paged: lane i holds the page of table column win_base + i
     for (int h = 0; h < n && live; ++h) {
       const int kb = w + 2 * h, sl = h % 3;
       const bool pre = kb < nb_pre;
@@ -296,6 +297,23 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
       const int count = min(kT5Keys, (pre ? prefix_len : own_keys) - j0);
       const bool tma = !pre || (prefix_tma && count == kT5Keys);
       const int row = pre ? prefix_start + j0 : seq_start + j0;
+      int ids[4] = {0, 0, 0, 0};  // paged: the pages of this block's (up to four) boxes of rows
+      if constexpr (kPaged) {
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          if (x * pg.box_rows >= count) break;
+          const int col = (j0 + x * pg.box_rows) / pg.c.P;
+          if (win_base < 0 || col < win_base || col >= win_base + 32) {
+            win_base = col & ~31;
+            win_id = win_base + lane < pg.c.max_pages ? pg.c.table[(long long)seq * pg.c.table_stride + win_base + lane] : -1;
+          }
+          ids[x] = __shfl_sync(0xffffffffu, win_id, col - win_base);
+          if (ids[x] < 0 || ids[x] >= pg.c.num_pages) {  // reported, and page 0 read in its place
+            if (lane == 0 && status) atomicOr(status, col < pg.c.max_pages ? B200KV_S_BAD_PAGE : B200KV_S_BAD_POSITION);
+            ids[x] = 0;
+          }
+        }
+      }
       for (int is_v = 0; is_v < 2 && live; ++is_v) {
         const uint32_t dst = (is_v ? ring_v(w) : ring_k(w)) + sl * kT5KvBytes;
         const uint32_t full = is_v ? bar_vf(w, sl) : bar_kf(w, sl), empty = is_v ? bar_ve(w, sl) : bar_ke(w, sl);
@@ -308,10 +326,10 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
             if (lane == 0) {
               const int R = pg.box_rows, nbox = (count + R - 1) / R;
               t5_mbar_expect_tx(full, (uint32_t)(nbox * R * 128 * blocks));
-              for (int x = 0; x < nbox; ++x) {
-                const int pos = j0 + x * R;
-                const int page = max(dec_page(pg.c, seq, pos, status), 0);  // a bad page is reported and page 0 read
-                const int prow = pos % pg.c.P, ph = page * pg.c.heads + hk;
+#pragma unroll
+              for (int x = 0; x < 4; ++x) {
+                if (x >= nbox) break;
+                const int prow = (j0 + x * R) % pg.c.P, ph = ids[x] * pg.c.heads + hk;
                 for (int bl = 0; bl < blocks; ++bl)
                   t5_tma_3d(dst + bl * (kT5Keys * 128) + x * R * 128, is_v ? &tm_v : &tm_k, 64 * bl, prow, ph, full);
               }
@@ -323,7 +341,7 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
               const bool valid = r < count && col < cols;
               const uint16_t* src = (const uint16_t*)pg.c.v;
               if (valid) {
-                const int page = max(dec_page(pg.c, seq, j0 + r, nullptr), 0);
+                const int x = r / pg.box_rows, page = x == 0 ? ids[0] : (x == 1 ? ids[1] : (x == 2 ? ids[2] : ids[3]));
                 src += dec_row(pg.c, page, hk, (j0 + r) % pg.c.P) * pg.c.v_row + col * 8;
               }
               t5_cp16(dst + (col >> 3) * (kT5Keys * 128) + r * 128 + (((col & 7) ^ (r & 7)) << 4), src, valid ? 16 : 0);

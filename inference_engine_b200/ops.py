@@ -268,15 +268,12 @@ def make_experts(router, gates, ups, downs, top: int, limit: float, slope: float
 
 
 def expert_tile_rows(num_rows: int, top: int, experts: int, dtype) -> int:
-    """Most rows of an expert's tile: up to 256 for prompt-sized steps (the widest tcgen05 tile; 128 when that leaves few
-    tiles to spread over the GPU), 64 for small ones, where weights are streamed and a narrow tile leaves shared memory
-    for a deeper ring."""
+    """Most rows of an expert's tile: 256 for prompt-sized steps (the widest tcgen05 tile), 64 for small ones, where
+    weights are streamed and a narrow tile leaves shared memory for a deeper ring."""
     if dtype == torch.float32:
         return 32
     total = num_rows * top
-    if total <= 512 or total <= 48 * experts:
-        return 64
-    return 128 if total <= 4096 else 256
+    return 64 if total <= 512 or total <= 48 * experts else 256
 
 
 def max_expert_tiles(total: int, experts: int, tile_rows: int) -> int:
