@@ -107,6 +107,109 @@ int b200dec_grouped_linear(const void* x, const void* w, int32_t elem, const int
                            int32_t total_rows, int32_t experts, int32_t out_rows, int32_t width, const float* score_sorted,
                            int32_t act, float limit, float slope, void* y, int32_t sm_count, int32_t variant, int32_t* status, void* stream);
 
+/* ---- attention with a sliding window, a sink and an output gate: the three kernels above with options.
+ * window > 0: the row at position i sees positions j with 0 <= i - j < window (0: all j <= i).
+ * sink fp32 [heads] (may be NULL): exp(sink[h]) joins the softmax denominator of head h, unscaled.
+ * gate (may be NULL), element size as the cache's: head h of row r is multiplied by sigmoid(gate[r * gate_stride + h]).
+ * out_scale multiplies the result; out rows are out_stride elements apart (0: heads * v_dim; a multiple of 8 otherwise). */
+typedef struct b200dec_attn_options {
+  int32_t window;
+  const float* sink;
+  const void* gate;
+  int64_t gate_stride;
+  float out_scale;
+  int64_t out_stride;
+} b200dec_attn_options;
+
+int b200dec_attn_rows_opt(const void* q, const b200dec_cache* cache, const b200kv_table* table, const b200dec_rows* rows, int32_t heads,
+                          float scale, const b200dec_attn_options* opt, void* out, int32_t* status, void* stream);
+int b200dec_decode_attn_opt(const void* q, const b200dec_cache* cache, const b200kv_table* table, const int32_t* cached_lens,
+                            const int32_t* num_decoding, int32_t B, int32_t heads, float scale, const b200dec_attn_options* opt, void* out,
+                            int32_t zero_idle, void* workspace, size_t workspace_bytes, int32_t sm_count, int32_t* status, void* stream);
+int b200dec_prefill_attn_opt(const void* q, const b200dec_cache* cache, const b200kv_table* table, const int32_t* seq_ids,
+                             const int32_t* cu_seqlens, const int32_t* cached_lens, const int32_t* tile_start, int32_t num_tiles,
+                             int32_t block_m, int32_t num_rows, int32_t heads, float scale, const b200dec_attn_options* opt, void* out,
+                             int32_t* status, void* stream);
+
+/* RMS norm of the whole query projection and of the whole key projection (q_norm fp32 [heads * k_dim], k_norm fp32
+ * [kv_heads * k_dim]), then rotary positions on channel pairs (2i, 2i + 1), i < half, then the write as in b200dec_rope_write
+ * (write_kv = 1).  cos_sin as there. */
+int b200dec_norm_rope_write(const void* qkv, int64_t qkv_stride, const b200dec_rows* rows, const b200dec_cache* cache,
+                            const b200kv_table* table, const float* q_norm, const float* k_norm, float eps, const float* cos_sin,
+                            int32_t table_len, int32_t half, int32_t heads, void* q_out, int32_t* status, void* stream);
+
+/* Residual update with the norm on the sublayer's output: x[r] += mult * (y[r] / sqrt(mean(y[r]^2) + eps) * weight), 32-bit;
+ * xb (may be NULL) receives the new row in the model's precision.  y has element size `elem`. */
+int b200dec_norm_add(float* x, const void* y, int32_t elem, const float* weight, float mult, float eps, void* xb, int32_t num_rows,
+                     int32_t width, void* stream);
+
+/* out[r, c] = silu(gate_up[r, c]) * gate_up[r, ff + c] */
+int b200dec_silu_mul(const void* gate_up, int64_t stride, int32_t elem, void* out, int64_t out_stride, int32_t num_rows, int32_t ff,
+                     void* stream);
+
+/* ---- recurrent layers: a matrix state per request slot and head, 32-bit.
+ * One token of one head (query/key head of head h: h / (heads / qk_heads)):
+ *   S <- decay * S;  u = beta (v - S^T k)  [correct]  or  step * v;  S <- S + k u^T;  o = S^T q (+ skip v)
+ * q, k, v pass a causal convolution of `taps` taps per channel and silu first; with unit_norm q and k are then divided by
+ * sqrt(sum(.^2) + unit_eps); q is multiplied by q_scale.  step = softplus(step_in + dt_bias), decay = exp(neg_a[h] step):
+ * one per head, or with channel_decay one per head and key channel (the rows of S); beta = sigmoid(beta_in).
+ * state fp32 [num_slots, heads, dim, round4(vdim)]; ring [num_slots, taps, channels] (element size elem): the convolution's
+ * raw inputs, position p at p % taps.  A request at position 0 starts from zero whatever its slot holds. */
+typedef struct b200dec_recurrence {
+  float* state;
+  void* ring;
+  const float* conv_w; /* [taps, channels], last row: the current token */
+  const float* conv_b; /* [channels] or NULL */
+  const float* neg_a;  /* [heads] */
+  const float* dt_bias; /* [heads], or [heads * dim] with channel_decay */
+  const float* skip;   /* [heads] or NULL */
+  int32_t num_slots, heads, qk_heads, dim, vdim, taps, elem;
+  int32_t channels, off_q, off_k, off_v; /* first convolution channel of q, k [qk_heads * dim] and v [heads * vdim] */
+  int32_t channel_decay, correct, unit_norm;
+  float unit_eps, q_scale;
+} b200dec_recurrence;
+
+/* A step's projection rows: x [channels] (the convolution's inputs), step [heads or heads * dim], beta [heads] (NULL without
+ * `correct`), row strides in elements. */
+typedef struct b200dec_recurrence_in {
+  const void* x;
+  const void* step;
+  const void* beta;
+  int64_t x_stride, step_stride, beta_stride;
+} b200dec_recurrence_in;
+
+/* A step's entries: rows cu_seqlens[e] .. cu_seqlens[e + 1] of entry e, which continues slot slots[e] at position
+ * cached_lens[e]; the first *num_decoding entries bring one token each.  cu_seqlens, seq_ids, positions NULL: pure decode,
+ * row e = entry e.  An entry with slot -1 (padding of a step) is passed over; its output rows are left as they are. */
+typedef struct b200dec_entries {
+  const int32_t* cu_seqlens;
+  const int32_t* cached_lens;
+  const int32_t* num_decoding;
+  const int32_t* slots;
+  const int32_t* seq_ids;
+  const int32_t* positions;
+  int32_t num_entries, num_rows;
+} b200dec_entries;
+
+/* The first *num_decoding rows, convolution and state in one kernel.  norm_w NULL: out fp32 [rows, heads * vdim] = o.
+ * Otherwise out (element size elem, row stride out_stride) = o / sqrt(mean over vdim(o^2) + eps) * norm_w[vdim] *
+ * sigmoid(gate) with gate rows [heads * vdim].  Rows from *num_decoding on of a pure decode step are zeroed. */
+int b200dec_recurrence_decode(const b200dec_recurrence* rec, const b200dec_recurrence_in* in, const b200dec_entries* ent,
+                              const float* norm_w, float eps, const void* gate, int64_t gate_stride, void* out, int64_t out_stride,
+                              int32_t* status, void* stream);
+/* Rows from *num_decoding on: silu(convolution) of every channel, conv_out [rows, channels rounded up to 8]. */
+int b200dec_conv_rows(const b200dec_recurrence* rec, const b200dec_recurrence_in* in, const b200dec_entries* ent, void* conv_out,
+                      int32_t* status, void* stream);
+/* Entries from *num_decoding on, token after token from conv_out: out fp32 [rows, heads * vdim]; the slots' states and rings
+ * are left at the portions' ends.  dim <= 1024. */
+int b200dec_recurrence_scan(const b200dec_recurrence* rec, const b200dec_recurrence_in* in, const void* conv_out,
+                            const b200dec_entries* ent, float* out, int32_t* status, void* stream);
+/* out[r] (element size elem) = out_scale * norm(o[r] (* silu(gate)  if gate_first)) * weight (* sigmoid(gate) otherwise), the norm
+ * taken over `parts` equal parts of the row of `len` each by itself; weight fp32 [weight_len], repeated.  */
+int b200dec_gated_norm(const float* o, const void* gate, int64_t gate_stride, int32_t gate_first, int32_t elem, const float* weight,
+                       int32_t weight_len, float eps, float out_scale, void* out, int64_t out_stride, int32_t num_rows, int32_t len,
+                       int32_t parts, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

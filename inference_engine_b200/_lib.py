@@ -44,8 +44,38 @@ class DecRows(C.Structure):
                 ("num_rows", c_int32)]
 
 
+class AttnOptions(C.Structure):
+    """struct b200dec_attn_options"""
+
+    _fields_ = [("window", c_int32), ("sink", c_void_p), ("gate", c_void_p), ("gate_stride", c_int64), ("out_scale", c_float),
+                ("out_stride", c_int64)]
+
+
+class Recurrence(C.Structure):
+    """struct b200dec_recurrence"""
+
+    _fields_ = [(n, c_void_p) for n in ("state", "ring", "conv_w", "conv_b", "neg_a", "dt_bias", "skip")] + [
+        (n, c_int32) for n in ("num_slots", "heads", "qk_heads", "dim", "vdim", "taps", "elem", "channels", "off_q", "off_k", "off_v",
+                               "channel_decay", "correct", "unit_norm")] + [("unit_eps", c_float), ("q_scale", c_float)]
+
+
+class RecurrenceIn(C.Structure):
+    """struct b200dec_recurrence_in"""
+
+    _fields_ = [("x", c_void_p), ("step", c_void_p), ("beta", c_void_p), ("x_stride", c_int64), ("step_stride", c_int64),
+                ("beta_stride", c_int64)]
+
+
+class Entries(C.Structure):
+    """struct b200dec_entries"""
+
+    _fields_ = [(n, c_void_p) for n in ("cu_seqlens", "cached_lens", "num_decoding", "slots", "seq_ids", "positions")] + [
+        ("num_entries", c_int32), ("num_rows", c_int32)]
+
+
 P_CACHE, P_TABLE = C.POINTER(Cache), C.POINTER(Table)
-P_DCACHE, P_ROWS = C.POINTER(DecCache), C.POINTER(DecRows)
+P_DCACHE, P_ROWS, P_OPT = C.POINTER(DecCache), C.POINTER(DecRows), C.POINTER(AttnOptions)
+P_REC, P_REC_IN, P_ENT = C.POINTER(Recurrence), C.POINTER(RecurrenceIn), C.POINTER(Entries)
 
 # name -> (restype, argtypes); must list every function include/b200kv.h declares
 SIGNATURES = {
@@ -113,6 +143,21 @@ DECODER_SIGNATURES = {
                                       c_void_p, c_size_t, c_int32, c_void_p, c_void_p]),
     "b200dec_prefill_attn": (c_int32, [c_void_p, P_DCACHE, P_TABLE, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
                                        c_int32, c_float, c_void_p, c_void_p, c_void_p]),
+    "b200dec_attn_rows_opt": (c_int32, [c_void_p, P_DCACHE, P_TABLE, P_ROWS, c_int32, c_float, P_OPT, c_void_p, c_void_p, c_void_p]),
+    "b200dec_decode_attn_opt": (c_int32, [c_void_p, P_DCACHE, P_TABLE, c_void_p, c_void_p, c_int32, c_int32, c_float, P_OPT, c_void_p,
+                                          c_int32, c_void_p, c_size_t, c_int32, c_void_p, c_void_p]),
+    "b200dec_prefill_attn_opt": (c_int32, [c_void_p, P_DCACHE, P_TABLE, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32,
+                                           c_int32, c_float, P_OPT, c_void_p, c_void_p, c_void_p]),
+    "b200dec_norm_rope_write": (c_int32, [c_void_p, c_int64, P_ROWS, P_DCACHE, P_TABLE, c_void_p, c_void_p, c_float, c_void_p, c_int32,
+                                          c_int32, c_int32, c_void_p, c_void_p, c_void_p]),
+    "b200dec_norm_add": (c_int32, [c_void_p, c_void_p, c_int32, c_void_p, c_float, c_float, c_void_p, c_int32, c_int32, c_void_p]),
+    "b200dec_silu_mul": (c_int32, [c_void_p, c_int64, c_int32, c_void_p, c_int64, c_int32, c_int32, c_void_p]),
+    "b200dec_recurrence_decode": (c_int32, [P_REC, P_REC_IN, P_ENT, c_void_p, c_float, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
+                                            c_void_p]),
+    "b200dec_conv_rows": (c_int32, [P_REC, P_REC_IN, P_ENT, c_void_p, c_void_p, c_void_p]),
+    "b200dec_recurrence_scan": (c_int32, [P_REC, P_REC_IN, c_void_p, P_ENT, c_void_p, c_void_p, c_void_p]),
+    "b200dec_gated_norm": (c_int32, [c_void_p, c_void_p, c_int64, c_int32, c_int32, c_void_p, c_int32, c_float, c_float, c_void_p, c_int64,
+                                     c_int32, c_int32, c_int32, c_void_p]),
     "b200dec_router": (c_int32, [c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p, c_void_p, c_void_p,
                                  c_void_p]),
     "b200dec_dispatch": (c_int32, [c_void_p, c_int32, c_void_p, c_void_p, c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_int32,

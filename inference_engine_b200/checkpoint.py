@@ -47,8 +47,28 @@ class Weights:
         self.taken.add(name)
         return t
 
+    def shape(self, name: str, default: tuple[int, ...]) -> tuple[int, ...]:
+        """Shape of a tensor whose sizes the configuration does not give (`default` where weights are made up)."""
+        if name not in self.tensors:
+            raise KeyError(f"the checkpoint has no tensor {name!r}")
+        return tuple(self.tensors[name].shape)
+
     def unused(self) -> list[str]:
         return sorted(set(self.tensors) - self.taken)
+
+
+class RandomWeights:
+    """Stand-in for a checkpoint: matrices ~ N(0, 1 / fan-in), norms near 1, drawn on the device."""
+
+    def __init__(self, device, seed: int = 0):
+        self.device, self.g = device, torch.Generator(device=device).manual_seed(seed)
+
+    def take(self, name: str, *shape: int) -> torch.Tensor:
+        t = torch.randn(*shape, generator=self.g, device=self.device)
+        return (1.0 + 0.1 * t if len(shape) == 1 else t * shape[-1] ** -0.5).to(torch.bfloat16)
+
+    def shape(self, name: str, default: tuple[int, ...]) -> tuple[int, ...]:
+        return default
 
 
 def read_safetensors(path: str) -> dict[str, torch.Tensor]:

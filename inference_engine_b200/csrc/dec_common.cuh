@@ -46,6 +46,10 @@ __device__ __forceinline__ float warp_sum(float v) {
   return v;
 }
 
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return fmaxf(z, 0.f) + log1pf(expf(-fabsf(z))); }
+
 // Device view of a b200dec_cache with its page table.
 struct DecCache {
   void* k;
@@ -84,6 +88,35 @@ inline int check_dec_cache(const b200dec_cache* c, const b200kv_table* t) {
   if (c->elem != 2 && c->elem != 4) return B200KV_E_SHAPE;
   if (t->max_pages < 1 || t->stride < 0) return B200KV_E_SHAPE;
   if (!aligned(c->k, 16) || !aligned(c->v, 16)) return B200KV_E_ALIGN;
+  return B200KV_OK;
+}
+
+// Device view of b200dec_attn_options (defaults filled in).
+struct DecAttnOpt {
+  int window;
+  const float* sink;
+  const void* gate;
+  long long gate_stride, out_stride;
+  float out_scale;
+  // what the finished output of (row, head) is multiplied by
+  template <typename T>
+  __device__ __forceinline__ float factor(long long r, int h) const {
+    return gate ? out_scale * sigmoid_f(ld_elem((const T*)gate + r * gate_stride + h)) : out_scale;
+  }
+};
+inline int dec_attn_opt(const b200dec_attn_options* o, int heads, int v_dim, DecAttnOpt* d) {
+  *d = DecAttnOpt{0, nullptr, nullptr, 0, (long long)heads * v_dim, 1.f};
+  if (!o) return B200KV_OK;
+  d->window = o->window;
+  d->sink = o->sink;
+  d->gate = o->gate;
+  d->gate_stride = o->gate_stride;
+  d->out_scale = o->out_scale;
+  if (o->window < 0) return B200KV_E_SHAPE;
+  if (o->out_stride) {
+    if (o->out_stride < d->out_stride || o->out_stride % 8) return B200KV_E_SHAPE;
+    d->out_stride = o->out_stride;
+  }
   return B200KV_OK;
 }
 

@@ -9,6 +9,8 @@
 // sums (query heads are the 16 rows of the product).  When the CTA's part of an (entry, head) ends, the four warps are
 // added up in shared memory; a part that is the whole of it is written out, otherwise it goes to the workspace and the
 // CTA that delivers the last part adds them (arrival counters return to zero).
+// With a sliding window only the blocks that hold a visible key are units; a sink joins the softmax sum when an (entry,
+// head) is complete, and the output gate multiplies there.
 // Every wait is bounded: when one runs out the CTA goes on without waiting, writes nothing and sets B200KV_S_TIMEOUT.
 #include "dec_tma.cuh"
 
@@ -56,6 +58,13 @@ __device__ __forceinline__ int pd_arrive(int* addr) {  // release my stores, acq
   return old;
 }
 
+// First block of 64 keys that a query at position len (its own key the last) sees, and the number of such blocks.
+__device__ __forceinline__ int pd_first(int len, int window) { return window > 0 ? max(0, len - window + 1) / kPdKeys : 0; }
+__device__ __forceinline__ int pd_blocks(int len, int window) {
+  len = max(len, 0);
+  return (len + kPdKeys) / kPdKeys - pd_first(len, window);
+}
+
 // Position in the flattened (entry, head unit, block) list.
 struct PdCursor {
   int b, hu, blk, nb, n;  // n: keys of the entry
@@ -88,8 +97,8 @@ struct PdCursor {
 template <int KB, int VB, bool kWide>
 __global__ void __launch_bounds__(kPdThreads, kPdCtasPerSm)
 paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* __restrict__ cached_lens,
-                    const int32_t* __restrict__ num_decoding, int B, int heads, int groups, float scale_log2, uint16_t* __restrict__ out,
-                    int zero_idle, int* __restrict__ counters, float* __restrict__ parts, int box_rows, int32_t* status,
+                    const int32_t* __restrict__ num_decoding, int B, int heads, int groups, float scale_log2, DecAttnOpt opt,
+                    uint16_t* __restrict__ out, int zero_idle, int* __restrict__ counters, float* __restrict__ parts, int box_rows, int32_t* status,
                     const __grid_constant__ CUtensorMap tm_k, const __grid_constant__ CUtensorMap tm_v) {
   extern __shared__ uint8_t pd_raw[];
   constexpr int kStages = pd_stages(KB, VB);
@@ -112,7 +121,7 @@ paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* _
   {
     const int chunk = (B + kPdThreads - 1) / kPdThreads, lo = min(tid * chunk, B), hi = min(lo + chunk, B);
     int sum = 0;
-    for (int b = lo; b < hi; ++b) sum += b < nd ? (max(cached_lens[b], 0) + kPdKeys) / kPdKeys : 0;
+    for (int b = lo; b < hi; ++b) sum += b < nd ? pd_blocks(cached_lens[b], opt.window) : 0;
     sums[tid] = sum;
     if (tid == 0) {
       for (int s = 0; s < kStages; ++s) {
@@ -142,7 +151,7 @@ paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* _
     int run = sums[tid];
     for (int b = lo; b < hi; ++b) {
       pre[b] = run;
-      run += b < nd ? (max(cached_lens[b], 0) + kPdKeys) / kPdKeys : 0;
+      run += b < nd ? pd_blocks(cached_lens[b], opt.window) : 0;
     }
     __syncthreads();
   }
@@ -150,7 +159,7 @@ paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* _
   if (zero_idle) {
     const int row = heads * c.v_dim;
     for (int b = nd + blockIdx.x; b < B; b += gridDim.x)
-      for (int i = tid; i < row; i += kPdThreads) out[(long long)b * row + i] = 0;
+      for (int i = tid; i < row; i += kPdThreads) out[b * opt.out_stride + i] = 0;
   }
   const int HU = c.heads * groups, total = HU * pre[B];
   const int per = max((total + (int)gridDim.x - 1) / (int)gridDim.x, kPdMinBlocks);
@@ -168,7 +177,8 @@ paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* _
       for (int u = u0; u < u1 && live; ++u, ++i) {
         const int s = i % kStages;
         if (i >= kStages && !dt_mbar_wait(empty(s), (i / kStages - 1) & 1)) { live = false; break; }
-        const int key0 = cur.blk * kPdKeys, nbox = (min(kPdKeys, cur.n - key0) + box_rows - 1) / box_rows;
+        const int key0 = (pd_first(cur.n - 1, opt.window) + cur.blk) * kPdKeys;
+        const int nbox = (min(kPdKeys, cur.n - key0) + box_rows - 1) / box_rows;
         const int hk = cur.hu / groups;
         dt_expect_tx(full(s), (uint32_t)nbox * box_rows * 128 * (KB + VB));
         const uint32_t dst = stage0 + s * kStageBytes;
@@ -205,6 +215,7 @@ paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* _
     const int head0 = hk * G + gq * kPdRows, nh = min(kPdRows, G - gq * kPdRows);
     const int ublk = cur.blk, nblk = min(cur.nb - cur.blk, u1 - u);
     const bool whole = ublk == 0 && nblk == cur.nb;
+    const int lo = opt.window > 0 ? max(0, cur.n - opt.window) : 0, blk0 = pd_first(cur.n - 1, opt.window) + ublk;
     uint32_t qa[4 * KB][4];
     {
       const uint16_t* r0 = q + ((long long)cur.b * heads + head0 + g) * c.k_row;
@@ -225,8 +236,9 @@ paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* _
     for (int k = 0; k < nblk; ++k, ++i) {
       const int s = i % kStages;
       if (!dead && !dt_mbar_wait(full(s), (i / kStages) & 1)) dead = true;
-      const int nvalid = cur.n - (ublk + k) * kPdKeys - warp * 16;  // keys of this warp's tile
-      if (nvalid > 0 && !dead) {
+      const int nvalid = cur.n - (blk0 + k) * kPdKeys - warp * 16;  // keys of this warp's tile
+      const int nskip = lo - (blk0 + k) * kPdKeys - warp * 16;      // ... and those in front of the window
+      if (nvalid > 0 && nskip < 16 && !dead) {
         const uint32_t sk = stage0 + s * kStageBytes, sv = sk + KB * kPdBlockBytes;
         float sc[2][4];
 #pragma unroll
@@ -245,7 +257,8 @@ paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* _
         for (int j = 0; j < 2; ++j)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            const bool in = 8 * j + 2 * t + e < nvalid;
+            const int key = 8 * j + 2 * t + e;
+            const bool in = key < nvalid && key >= nskip;
             sc[j][e] = in ? sc[j][e] * scale_log2 : -INFINITY;
             mx0 = fmaxf(mx0, sc[j][e]);
             if (kWide) {
@@ -319,7 +332,18 @@ paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* _
       M0 = fmaxf(M0, ml[w][g][0]);
       M1 = fmaxf(M1, ml[w][g + 8][0]);
     }
+    float sink0 = -INFINITY, sink1 = -INFINITY;
+    if (whole && opt.sink) {
+      if (g < nh) sink0 = opt.sink[head0 + g] * 1.4426950408889634f;
+      if (kWide && g + 8 < nh) sink1 = opt.sink[head0 + g + 8] * 1.4426950408889634f;
+      M0 = fmaxf(M0, sink0);
+      M1 = fmaxf(M1, sink1);
+    }
     const float B0 = M0 == -INFINITY ? 0.f : M0, B1 = M1 == -INFINITY ? 0.f : M1;
+    if (whole && opt.sink) {
+      L0 = pd_exp2(sink0 - B0);
+      L1 = pd_exp2(sink1 - B1);
+    }
 #pragma unroll
     for (int w = 0; w < kPdWarps; ++w) {
       L0 += ml[w][g][1] * pd_exp2(ml[w][g][0] - B0);
@@ -350,11 +374,12 @@ paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* _
     }
     const bool lost = *(volatile int*)&flag_dead != 0;
     if (lost && status && tid == 0) atomicOr(status, B200KV_S_TIMEOUT);
-    const long long orow = ((long long)cur.b * heads + head0) * c.v_dim;
+    const long long orow = cur.b * opt.out_stride + head0 * c.v_dim;
     if (whole) {
       if (warp == 0 && !lost) {
-        const float i0 = L0 > 0.f ? 1.f / L0 : 0.f, i1 = L1 > 0.f ? 1.f / L1 : 0.f;
-        const bool pairs = c.v_dim % 2 == 0;
+        const float i0 = (L0 > 0.f ? 1.f / L0 : 0.f) * (g < nh ? opt.factor<uint16_t>(cur.b, head0 + g) : 0.f);
+        const float i1 = (L1 > 0.f ? 1.f / L1 : 0.f) * (kWide && g + 8 < nh ? opt.factor<uint16_t>(cur.b, head0 + g + 8) : 0.f);
+        const bool pairs = c.v_dim % 2 == 0 && opt.out_stride % 2 == 0;
 #pragma unroll
         for (int j = 0; j < kTiles; ++j)
 #pragma unroll
@@ -398,20 +423,21 @@ paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* _
         for (int x = tid; x < nh * 64 * VB; x += 32 * kPdWarps) {
           const int row = x / (64 * VB), ch = x - row * (64 * VB);
           if (ch >= c.v_dim) continue;
-          float M = -INFINITY;
+          const float sink = opt.sink ? opt.sink[head0 + row] * 1.4426950408889634f : -INFINITY;
+          float M = sink;
           for (int cc = c_lo; cc <= c_hi; ++cc) {
             const float* p = parts + (long long)(2 * cc + (a <= cc * per ? 0 : 1)) * kPart;
             M = fmaxf(M, __ldcg(p + kPdRows * 64 * VB + row));
           }
           const float base = M == -INFINITY ? 0.f : M;
-          float L = 0.f, acc = 0.f;
+          float L = opt.sink ? pd_exp2(sink - base) : 0.f, acc = 0.f;
           for (int cc = c_lo; cc <= c_hi; ++cc) {
             const float* p = parts + (long long)(2 * cc + (a <= cc * per ? 0 : 1)) * kPart;
             const float f = pd_exp2(__ldcg(p + kPdRows * 64 * VB + row) - base);
             L = fmaf(f, __ldcg(p + kPdRows * 64 * VB + kPdRows + row), L);
             acc = fmaf(f, __ldcg(p + row * (64 * VB) + ch), acc);
           }
-          st_elem(out + orow + (long long)row * c.v_dim + ch, L > 0.f ? acc / L : 0.f);
+          st_elem(out + orow + (long long)row * c.v_dim + ch, L > 0.f ? acc / L * opt.factor<uint16_t>(cur.b, head0 + row) : 0.f);
         }
         if (tid == 0) counters[cur.b * HU + cur.hu] = 0;
       }
@@ -424,13 +450,13 @@ paged_decode_kernel(const uint16_t* __restrict__ q, DecCache c, const int32_t* _
 
 template <int KB, int VB, bool kWide>
 static int pd_launch(const void* q, const DecCache& c, const int32_t* cached_lens, const int32_t* num_decoding, int B, int heads, int groups,
-                     float scale_log2, void* out, int zero_idle, int* counters, float* parts, int grid, int box_rows, int32_t* status,
+                     float scale_log2, const DecAttnOpt& opt, void* out, int zero_idle, int* counters, float* parts, int grid, int box_rows, int32_t* status,
                      const CUtensorMap& tm_k, const CUtensorMap& tm_v, cudaStream_t stream) {
   const size_t smem = (size_t)pd_stages(KB, VB) * (KB + VB) * kPdBlockBytes + 1024 + (size_t)(B + 1) * 4;
   if (cudaFuncSetAttribute(paged_decode_kernel<KB, VB, kWide>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     return B200KV_E_LAUNCH;
   return launch_result(launch_chained(paged_decode_kernel<KB, VB, kWide>, dim3(grid), dim3(kPdThreads), smem, stream, (const uint16_t*)q, c,
-                                      cached_lens, num_decoding, B, heads, groups, scale_log2, (uint16_t*)out, zero_idle, counters, parts,
+                                      cached_lens, num_decoding, B, heads, groups, scale_log2, opt, (uint16_t*)out, zero_idle, counters, parts,
                                       box_rows, status, tm_k, tm_v));
 }
 
@@ -447,9 +473,10 @@ extern "C" size_t b200dec_decode_attn_workspace(int32_t B, int32_t heads, int32_
   return pd_counter_bytes(B, heads) + (size_t)sm_count * kPdCtasPerSm * 2 * kPdRows * (64 * vb + 2) * 4;
 }
 
-extern "C" int b200dec_decode_attn(const void* q, const b200dec_cache* cache, const b200kv_table* table, const int32_t* cached_lens,
-                                   const int32_t* num_decoding, int32_t B, int32_t heads, float scale, void* out, int32_t zero_idle,
-                                   void* workspace, size_t workspace_bytes, int32_t sm_count, int32_t* status, void* stream) {
+extern "C" int b200dec_decode_attn_opt(const void* q, const b200dec_cache* cache, const b200kv_table* table, const int32_t* cached_lens,
+                                       const int32_t* num_decoding, int32_t B, int32_t heads, float scale,
+                                       const b200dec_attn_options* options, void* out, int32_t zero_idle, void* workspace,
+                                       size_t workspace_bytes, int32_t sm_count, int32_t* status, void* stream) {
   if (B == 0) return B200KV_OK;
   if (!q || !cached_lens || !num_decoding || !out || !workspace) return B200KV_E_NULL;
   const int rc = check_dec_cache(cache, table);
@@ -459,6 +486,9 @@ extern "C" int b200dec_decode_attn(const void* q, const b200dec_cache* cache, co
   if (B < 0 || B > kPdMaxB || sm_count < 1 || (long long)cache->num_pages * cache->kv_heads > 0x7FFFFFFFll ||
       (long long)B * heads * table->max_pages * ((cache->page_size + kPdKeys - 1) / kPdKeys) > 0x3FFFFFFFll)
     return B200KV_E_RANGE;
+  DecAttnOpt opt;
+  const int bad = dec_attn_opt(options, heads, cache->v_dim, &opt);
+  if (bad != B200KV_OK) return bad;
   if (!aligned(q, 16) || !aligned(out, 4) || !aligned(workspace, 256)) return B200KV_E_ALIGN;
   if (workspace_bytes < b200dec_decode_attn_workspace(B, heads, cache->kv_heads, cache->v_dim, sm_count)) return B200KV_E_WORKSPACE;
   const DecCache c = dec_view(cache, table);
@@ -470,7 +500,9 @@ extern "C" int b200dec_decode_attn(const void* q, const b200dec_cache* cache, co
   int* counters = (int*)workspace;
   float* parts = (float*)((uint8_t*)workspace + pd_counter_bytes(B, heads));
   // no more CTAs than the largest batch the table can address has shares of the smallest size
-  const long long units = (long long)B * c.heads * groups * (((long long)c.max_pages * c.P + kPdKeys - 1) / kPdKeys);
+  long long entry_blocks = ((long long)c.max_pages * c.P + kPdKeys - 1) / kPdKeys;
+  if (opt.window > 0 && entry_blocks > opt.window / kPdKeys + 2) entry_blocks = opt.window / kPdKeys + 2;
+  const long long units = (long long)B * c.heads * groups * entry_blocks;
   const long long want = (units + kPdMinBlocks - 1) / kPdMinBlocks;
   const int grid = (int)(want < (long long)sm_count * kPdCtasPerSm ? want : (long long)sm_count * kPdCtasPerSm);
   const float sl = scale * 1.4426950408889634f;
@@ -478,10 +510,17 @@ extern "C" int b200dec_decode_attn(const void* q, const b200dec_cache* cache, co
   cudaStream_t s = (cudaStream_t)stream;
 #define PD_CASE(KB, VB, W)                                                                                                        \
   if (kb == KB - 1 && vb == VB - 1 && wide == W)                                                                                  \
-    return pd_launch<KB, VB, W>(q, c, cached_lens, num_decoding, B, heads, groups, sl, out, zero_idle, counters, parts, grid, box, \
+    return pd_launch<KB, VB, W>(q, c, cached_lens, num_decoding, B, heads, groups, sl, opt, out, zero_idle, counters, parts, grid, box, \
                                 status, tm_k, tm_v, s);
   PD_CASE(1, 1, false) PD_CASE(1, 1, true) PD_CASE(1, 2, false) PD_CASE(1, 2, true)
   PD_CASE(2, 1, false) PD_CASE(2, 1, true) PD_CASE(2, 2, false) PD_CASE(2, 2, true)
 #undef PD_CASE
   return B200KV_E_SHAPE;
+}
+
+extern "C" int b200dec_decode_attn(const void* q, const b200dec_cache* cache, const b200kv_table* table, const int32_t* cached_lens,
+                                   const int32_t* num_decoding, int32_t B, int32_t heads, float scale, void* out, int32_t zero_idle,
+                                   void* workspace, size_t workspace_bytes, int32_t sm_count, int32_t* status, void* stream) {
+  return b200dec_decode_attn_opt(q, cache, table, cached_lens, num_decoding, B, heads, scale, nullptr, out, zero_idle, workspace,
+                                 workspace_bytes, sm_count, status, stream);
 }

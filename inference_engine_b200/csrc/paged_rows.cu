@@ -1,4 +1,5 @@
-// The paged cache of unquantised rows: rotary positions + unit norm + write of keys and values (one kernel), and the
+// The paged cache of unquantised rows: rotary positions + unit norm + write of keys and values (one kernel; a second one
+// norms whole projections first and rotates neighbouring channels), and the
 // general attention over it (any sizes, bf16 or fp32, prompt portions and decoding alike) on the CUDA cores.
 #include "dec_common.cuh"
 
@@ -120,6 +121,119 @@ rope_write_kernel(const T* __restrict__ qkv, long long qkv_stride, b200dec_rows 
   }
 }
 
+// ---------------------------------------------------------------- norm of whole projections, interleaved rotation, write
+// One block per row.  kPairs: head sizes and the row stride are even, so channel pairs are loaded together.
+constexpr int kNrThreads = 256;
+
+template <typename T, bool kPairs>
+__global__ void __launch_bounds__(kNrThreads)
+norm_rope_write_kernel(const T* __restrict__ qkv, long long qkv_stride, b200dec_rows rows, DecCache c, const float* __restrict__ q_norm,
+                       const float* __restrict__ k_norm, float eps, const float* __restrict__ cos_sin, int table_len, int half, int heads,
+                       T* __restrict__ q_out, int32_t* status) {
+  __shared__ float part[2][kNrThreads / 32];
+  pdl_enter();
+  const int r = blockIdx.x, tid = threadIdx.x;
+  T* qdst = q_out + (long long)r * heads * c.k_row;
+  int seq = r, pos;
+  if (rows.seq_ids) {
+    seq = rows.seq_ids[r];
+    pos = rows.positions[r];
+  } else {
+    if (r >= *rows.num_decoding) {  // an idle row: nothing is written to the cache, q reads as zero
+      pdl_wait();
+      for (int ch = tid; ch < heads * c.k_row; ch += kNrThreads) st_elem(qdst + ch, 0.f);
+      return;
+    }
+    pos = rows.cached_lens[r];
+  }
+  const bool ok = pos >= 0 && (half == 0 || pos < table_len);
+  if (!ok) {
+    if (tid == 0 && status) atomicOr(status, B200KV_S_BAD_POSITION);
+    pos = 0;
+  }
+  const int page = ok ? dec_page(c, seq, pos, tid == 0 ? status : nullptr) : -1;
+  pdl_wait();
+  const T* src = qkv + r * qkv_stride;
+  const int nq = heads * c.k_dim, nk = c.heads * c.k_dim;
+  float sq = 0.f, sk = 0.f;
+  if (kPairs) {
+    for (int i = 2 * tid; i < nq + nk; i += 2 * kNrThreads) {
+      const float2 v = rw_load2(src + i);
+      const float s2 = fmaf(v.x, v.x, v.y * v.y);
+      if (i < nq) sq += s2; else sk += s2;
+    }
+  } else {
+    for (int i = tid; i < nq + nk; i += kNrThreads) {
+      const float v = ld_elem(src + i);
+      if (i < nq) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk);
+    }
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((tid & 31) == 0) {
+    part[0][tid >> 5] = sq;
+    part[1][tid >> 5] = sk;
+  }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < kNrThreads / 32; ++i) {
+    sq += part[0][i];
+    sk += part[1][i];
+  }
+  const float inv_q = 1.0f / sqrtf(sq / (float)nq + eps), inv_k = 1.0f / sqrtf(sk / (float)nk + eps);
+  const float2* cs = reinterpret_cast<const float2*>(cos_sin) + (long long)pos * half;
+  auto put2 = [](T* dst, float a, float b) {
+    if (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = float_to_bf16_bits(a) | (float_to_bf16_bits(b) << 16);
+    else *reinterpret_cast<float2*>(dst) = make_float2(a, b);
+  };
+  const int kpairs = c.k_row / 2, vpairs = c.v_row / 2;  // channels behind a size are written as zero
+  const long long at0 = page < 0 ? 0 : dec_row(c, page, 0, pos % c.P);
+  for (int i = tid; i < (heads + c.heads) * kpairs; i += kNrThreads) {
+    const int h = i / kpairs, pr = i - h * kpairs, ch = 2 * pr;
+    const bool is_q = h < heads;
+    if (!is_q && page < 0) continue;
+    float a = 0.f, b = 0.f;
+    if (ch < c.k_dim) {
+      const int off = h * c.k_dim + ch;  // q heads and k heads lie end to end
+      const float* w = is_q ? q_norm + off : k_norm + (off - nq);
+      const float inv = is_q ? inv_q : inv_k;
+      if (kPairs) {
+        const float2 v = rw_load2(src + off);
+        a = v.x * inv * w[0];
+        b = v.y * inv * w[1];
+      } else {
+        a = ld_elem(src + off) * inv * w[0];
+        if (ch + 1 < c.k_dim) b = ld_elem(src + off + 1) * inv * w[1];
+      }
+      if (pr < half) {
+        const float2 t = cs[pr];
+        const float u = a, v = b;
+        a = u * t.x - v * t.y;
+        b = v * t.x + u * t.y;
+      }
+    }
+    put2(is_q ? qdst + h * c.k_row + ch : (T*)c.k + (at0 + (long long)(h - heads) * c.P) * c.k_row + ch, a, b);
+  }
+  if (page < 0) return;
+  const T* vsrc = src + nq + nk;
+  for (int i = tid; i < c.heads * vpairs; i += kNrThreads) {
+    const int h = i / vpairs, ch = 2 * (i - h * vpairs);
+    float a = 0.f, b = 0.f;
+    if (ch < c.v_dim) {
+      if (kPairs) {
+        const float2 v = rw_load2(vsrc + h * c.v_dim + ch);
+        a = v.x;
+        b = v.y;
+      } else {
+        a = ld_elem(vsrc + h * c.v_dim + ch);
+        if (ch + 1 < c.v_dim) b = ld_elem(vsrc + h * c.v_dim + ch + 1);
+      }
+    }
+    put2((T*)c.v + (at0 + (long long)h * c.P) * c.v_row + ch, a, b);
+  }
+}
+
 // ---------------------------------------------------------------- attention, one block per (row, query head)
 constexpr int kArThreads = 128;
 constexpr int kArKeys = 128;  // keys per block step, one score per thread
@@ -127,7 +241,8 @@ constexpr int kArPieces = 8;  // channels of the output per thread: v_dim up to 
 
 template <typename T>
 __global__ void __launch_bounds__(kArThreads)
-attn_rows_kernel(const T* __restrict__ q, DecCache c, b200dec_rows rows, int heads, float scale, T* __restrict__ out, int32_t* status) {
+attn_rows_kernel(const T* __restrict__ q, DecCache c, b200dec_rows rows, int heads, float scale, DecAttnOpt opt, T* __restrict__ out,
+                 int32_t* status) {
   extern __shared__ float ar_smem[];
   float* qs = ar_smem;                                                  // [k_dim]
   float* ps = qs + ((c.k_dim + 3) / 4) * 4;                             // [kArKeys]
@@ -135,7 +250,7 @@ attn_rows_kernel(const T* __restrict__ q, DecCache c, b200dec_rows rows, int hea
   __shared__ float red[2][kArThreads / 32];
   pdl_enter();
   const int r = blockIdx.y, h = blockIdx.x, hk = h / (heads / c.heads), tid = threadIdx.x;
-  T* dst = out + ((long long)r * heads + h) * c.v_dim;
+  T* dst = out + r * opt.out_stride + h * c.v_dim;
   int seq = r, pos;
   if (rows.seq_ids) {
     seq = rows.seq_ids[r];
@@ -150,10 +265,10 @@ attn_rows_kernel(const T* __restrict__ q, DecCache c, b200dec_rows rows, int hea
   }
   const T* qrow = q + ((long long)r * heads + h) * c.k_row;
   for (int ch = tid; ch < c.k_dim; ch += kArThreads) qs[ch] = ld_elem(qrow + ch) * scale;
-  float m = -INFINITY, l = 0.f, o[kArPieces];
+  float m = opt.sink ? opt.sink[h] : -INFINITY, l = opt.sink ? 1.f : 0.f, o[kArPieces];
 #pragma unroll
   for (int i = 0; i < kArPieces; ++i) o[i] = 0.f;
-  for (int j0 = 0; j0 <= pos; j0 += kArKeys) {
+  for (int j0 = opt.window > 0 ? max(0, pos - opt.window + 1) : 0; j0 <= pos; j0 += kArKeys) {
     const int n = min(kArKeys, pos + 1 - j0);
     __syncthreads();
     int at = -1;
@@ -204,7 +319,7 @@ attn_rows_kernel(const T* __restrict__ q, DecCache c, b200dec_rows rows, int hea
       }
     }
   }
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  const float inv = (l > 0.f ? 1.f / l : 0.f) * opt.factor<T>(r, h);
 #pragma unroll
   for (int i = 0; i < kArPieces; ++i) {
     const int ch = tid + i * kArThreads;
@@ -254,12 +369,39 @@ extern "C" int b200dec_rope_write(const void* qkv, int64_t qkv_stride, const b20
   return run(pairs ? rope_write_kernel<float, true, kRwMaxPairs> : rope_write_kernel<float, false, kRwMaxPairs>, (const float*)qkv, (float*)q_out);
 }
 
-extern "C" int b200dec_attn_rows(const void* q, const b200dec_cache* cache, const b200kv_table* table, const b200dec_rows* rows,
-                                 int32_t heads, float scale, void* out, int32_t* status, void* stream) {
+extern "C" int b200dec_norm_rope_write(const void* qkv, int64_t qkv_stride, const b200dec_rows* rows, const b200dec_cache* cache,
+                                       const b200kv_table* table, const float* q_norm, const float* k_norm, float eps,
+                                       const float* cos_sin, int32_t table_len, int32_t half, int32_t heads, void* q_out, int32_t* status,
+                                       void* stream) {
+  if (rows && rows->num_rows == 0) return B200KV_OK;
+  if (!qkv || !q_out || !q_norm || !k_norm) return B200KV_E_NULL;
+  int rc = check_rows(rows);
+  if (rc == B200KV_OK) rc = check_dec_cache(cache, table);
+  if (rc != B200KV_OK) return rc;
+  if (half < 0 || 2 * half > cache->k_dim || (half > 0 && (!cos_sin || table_len < 1))) return B200KV_E_SHAPE;
+  if (heads < 1 || heads % cache->kv_heads) return B200KV_E_SHAPE;
+  if (!aligned(q_out, 16) || !aligned(cos_sin, 8)) return B200KV_E_ALIGN;
+  const DecCache c = dec_view(cache, table);
+  cudaStream_t s = (cudaStream_t)stream;
+  const bool pairs = cache->k_dim % 2 == 0 && cache->v_dim % 2 == 0 && qkv_stride % 2 == 0 && aligned(qkv, 2 * cache->elem);
+  auto run = [&](auto* kernel, auto* in, auto* q) {
+    return launch_result(launch_chained(kernel, dim3(rows->num_rows), dim3(kNrThreads), 0, s, in, (long long)qkv_stride, *rows, c, q_norm,
+                                        k_norm, eps, cos_sin, table_len, half, heads, q, status));
+  };
+  if (cache->elem == 2)
+    return run(pairs ? norm_rope_write_kernel<uint16_t, true> : norm_rope_write_kernel<uint16_t, false>, (const uint16_t*)qkv, (uint16_t*)q_out);
+  return run(pairs ? norm_rope_write_kernel<float, true> : norm_rope_write_kernel<float, false>, (const float*)qkv, (float*)q_out);
+}
+
+extern "C" int b200dec_attn_rows_opt(const void* q, const b200dec_cache* cache, const b200kv_table* table, const b200dec_rows* rows,
+                                     int32_t heads, float scale, const b200dec_attn_options* options, void* out, int32_t* status,
+                                     void* stream) {
   if (rows && rows->num_rows == 0) return B200KV_OK;
   if (!q || !out) return B200KV_E_NULL;
   int rc = check_rows(rows);
   if (rc == B200KV_OK) rc = check_dec_cache(cache, table);
+  DecAttnOpt opt;
+  if (rc == B200KV_OK) rc = dec_attn_opt(options, heads, cache->v_dim, &opt);
   if (rc != B200KV_OK) return rc;
   if (heads < 1 || heads % cache->kv_heads || cache->v_dim > kArThreads * kArPieces || cache->k_dim > 1024) return B200KV_E_SHAPE;
   if ((long long)cache->num_pages * cache->page_size > 0x7FFFFFFFll || rows->num_rows > 65535) return B200KV_E_RANGE;
@@ -268,7 +410,12 @@ extern "C" int b200dec_attn_rows(const void* q, const b200dec_cache* cache, cons
   cudaStream_t s = (cudaStream_t)stream;
   if (cache->elem == 2)
     return launch_result(launch_chained(attn_rows_kernel<uint16_t>, dim3(heads, rows->num_rows), dim3(kArThreads), smem, s,
-                                        (const uint16_t*)q, c, *rows, heads, scale, (uint16_t*)out, status));
+                                        (const uint16_t*)q, c, *rows, heads, scale, opt, (uint16_t*)out, status));
   return launch_result(launch_chained(attn_rows_kernel<float>, dim3(heads, rows->num_rows), dim3(kArThreads), smem, s, (const float*)q, c,
-                                      *rows, heads, scale, (float*)out, status));
+                                      *rows, heads, scale, opt, (float*)out, status));
+}
+
+extern "C" int b200dec_attn_rows(const void* q, const b200dec_cache* cache, const b200kv_table* table, const b200dec_rows* rows,
+                                 int32_t heads, float scale, void* out, int32_t* status, void* stream) {
+  return b200dec_attn_rows_opt(q, cache, table, rows, heads, scale, nullptr, out, status, stream);
 }

@@ -43,6 +43,8 @@
 // head size 128.  The paged one (kPaged = true, paged_prefill_tc5.cu) reads keys and values of the whole sequence, the
 // chunk's own included, by page from a cache of bf16 rows, with key and value sizes of up to 128 each: copies beyond a
 // size read as zero, products run over the blocks of 64 channels there are, and a query at position p sees keys 0..p.
+// With kOptions a sliding window leaves out the blocks in front of the tile's first row's window and masks the rest, a
+// sink is what the first warpgroup's softmax state starts from, and the output gate multiplies in the last step.
 //
 // Every wait on an mbarrier is bounded: if a completion never arrives the waiting role records it, stops
 // issuing work and the CTA skips its stores, sets B200KV_S_TIMEOUT in the status word, frees its tensor
@@ -176,9 +178,10 @@ struct T5Paged {
   DecCache c;
   const int32_t* cached_lens;
   int box_rows;
+  DecAttnOpt opt;
 };
 
-template <bool kPaged, int kKeyBlocks = 2>  // kKeyBlocks: 64-channel blocks of a key (2 covers up to 128 channels)
+template <bool kPaged, int kKeyBlocks = 2, bool kOptions = false>  // kKeyBlocks: 64-channel blocks of a key (2 covers up to 128 channels)
 __global__ void __launch_bounds__(kT5Threads, 1)
 prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long long q_sh, const uint16_t* __restrict__ k,
                         long long k_sn, long long k_sh, const uint16_t* __restrict__ v, long long v_sn, long long v_sh,
@@ -216,7 +219,9 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
   const int cta_last = min(row0 + kT5Tile, row_end) - 1;
   const int own_keys = cached + cta_last - seq_start + 1;  // causal: keys up to the CTA's last query
   const int nb_pre = (prefix_len + kT5Keys - 1) / kT5Keys, nb_own = (own_keys + kT5Keys - 1) / kT5Keys;
-  const int nb = nb_pre + nb_own;
+  // blocks in front of every row's window
+  const int skipped = kOptions && pg.opt.window > 0 ? max(0, cached + row0 - seq_start - pg.opt.window + 1) / kT5Keys : 0;
+  const int nb = nb_pre + nb_own - skipped;
 
   float m_ref_keep = -INFINITY, l_keep = 0.f;
   // roles: warps 0-3 and 4-7 = softmax warpgroups 0 and 1, warps 8 and 9 = issue the products of warpgroup 0
@@ -293,7 +298,7 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
     for (int h = 0; h < n && live; ++h) {
       const int kb = w + 2 * h, sl = h % 3;
       const bool pre = kb < nb_pre;
-      const int j0 = pre ? kb * kT5Keys : (kb - nb_pre) * kT5Keys;
+      const int j0 = pre ? kb * kT5Keys : (kb - nb_pre + skipped) * kT5Keys;
       const int count = min(kT5Keys, (pre ? prefix_len : own_keys) - j0);
       const bool tma = !pre || (prefix_tma && count == kT5Keys);
       const int row = pre ? prefix_start + j0 : seq_start + j0;
@@ -425,6 +430,17 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
     const int my_keys = min(own_keys, cached + row0 + wt - seq_start + 1);  // own-chunk keys this row may see
     const int first_keys = min(own_keys, cached + row0 - seq_start + 1);    // ... and the tile's first row
     float m_ref = -INFINITY, l = 0.f;  // offset of the exponentials (log2 units, scaled), running sum
+    int my_first = 0, last_first = 0;  // first key in the window of this row and of the tile's last row
+    if constexpr (kOptions) {
+      if (pg.opt.window > 0) {
+        my_first = cached + row0 + wt - seq_start - pg.opt.window + 1;
+        last_first = cached + cta_last - seq_start - pg.opt.window + 1;
+      }
+      if (pg.opt.sink && wg == 0) {
+        m_ref = pg.opt.sink[hq] * 1.4426950408889634f;
+        l = 1.f;
+      }
+    }
     bool ok = true;
     for (int h = 0; h < n_mine && ok; ++h) {
       ok = t5_mbar_wait(bar_s(wg, h & 1), (h >> 1) & 1, spin);  // S(h) is complete
@@ -432,9 +448,11 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
       // ---- softmax of this thread's row
       const int kb = wg + 2 * h;
       const bool pre = kb < nb_pre;
-      const int j0 = pre ? kb * kT5Keys : (kb - nb_pre) * kT5Keys;
+      const int j0 = pre ? kb * kT5Keys : (kb - nb_pre + skipped) * kT5Keys;
       const int lim = (pre ? prefix_len : my_keys) - j0;                // keys [0, lim) visible to this row
-      const bool full = (pre ? prefix_len : first_keys) - j0 >= kT5Keys;  // ... all 64 to every row of the tile
+      const int low = kOptions ? my_first - j0 : 0;                      // ... but for those in front of its window
+      // ... all 64 to every row of the tile
+      const bool full = (pre ? prefix_len : first_keys) - j0 >= kT5Keys && (!kOptions || last_first <= j0);
       uint32_t u[64];
       t5_ld64(tS + 64 * (h & 1), u);
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};  // four chains instead of one of 64
@@ -443,7 +461,7 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
         for (int c = 0; c < 64; ++c) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(u[c]));
       } else {
 #pragma unroll
-        for (int c = 0; c < 64; ++c) mx4[c & 3] = fmaxf(mx4[c & 3], c < lim ? __uint_as_float(u[c]) : -INFINITY);
+        for (int c = 0; c < 64; ++c) mx4[c & 3] = fmaxf(mx4[c & 3], c < lim && (!kOptions || c >= low) ? __uint_as_float(u[c]) : -INFINITY);
       }
       const float r = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;
       const bool move = r > m_ref + kT5Lazy;  // also true for the first visible key of a row (m_ref = -inf)
@@ -481,8 +499,8 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
       } else {
 #pragma unroll
         for (int c = 0; c < 32; ++c) {
-          const float p0 = 2 * c < lim ? t5_exp2(fmaf(__uint_as_float(u[2 * c]), scale_log2, -off)) : 0.f;
-          const float p1 = 2 * c + 1 < lim ? t5_exp2(fmaf(__uint_as_float(u[2 * c + 1]), scale_log2, -off)) : 0.f;
+          const float p0 = 2 * c < lim && (!kOptions || 2 * c >= low) ? t5_exp2(fmaf(__uint_as_float(u[2 * c]), scale_log2, -off)) : 0.f;
+          const float p1 = 2 * c + 1 < lim && (!kOptions || 2 * c + 1 >= low) ? t5_exp2(fmaf(__uint_as_float(u[2 * c + 1]), scale_log2, -off)) : 0.f;
           ps4[c & 3] += p0 + p1;
           pk[c] = t5_pack_bf16x2(p0, p1);
         }
@@ -536,7 +554,8 @@ prefill_attn_tc5_kernel(const uint16_t* __restrict__ q, long long q_sn, long lon
       const float mm = fmaxf(m0, m1);
       const float a0 = m0 == -INFINITY ? 0.f : t5_exp2(m0 - mm), a1 = m1 == -INFINITY ? 0.f : t5_exp2(m1 - mm);
       const float lt = l0 * a0 + l1 * a1;
-      const float inv = lt != 0.f ? 1.f / lt : 0.f;  // kernels.py:1118
+      float inv = lt != 0.f ? 1.f / lt : 0.f;  // kernels.py:1118
+      if constexpr (kOptions) inv *= my_row < row_end ? pg.opt.factor<uint16_t>(my_row, hq) : 0.f;
       const float f0 = a0 * inv, f1 = a1 * inv;
       uint4* dst = reinterpret_cast<uint4*>(out + (long long)my_row * o_sn + hq * o_sh);
 #pragma unroll

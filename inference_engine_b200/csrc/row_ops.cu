@@ -1,6 +1,7 @@
 // Row-wise ops of a decoder with a 32-bit residual stream: embedding rows, and the residual update of the
 // norm-after-the-sum arrangement with the optional sum over a token's experts.  HBM-bound streaming kernels; one
-// block per row, the row in registers between the two passes.
+// block per row, the row in registers between the two passes.  Also the arrangement with the norm on a sublayer's output,
+// the gated unit of a dense feed-forward, and the norm of a row's parts with a gate.
 #include "dec_common.cuh"
 
 namespace b200kv {
@@ -124,6 +125,150 @@ scaled_add_norm_any_kernel(const float* x, const T* __restrict__ delta, const in
   }
 }
 
+// x += mult * rmsnorm(y) * weight, one block per row.  kChunks > 0: y in registers between the passes (width % 4 == 0),
+// 0: any width, y is read twice.
+template <typename T, int kChunks>
+__global__ void __launch_bounds__(kRowThreads)
+norm_add_kernel(float* x, const T* __restrict__ y, const float* __restrict__ weight, float mult, float eps, T* __restrict__ xb, int width) {
+  pdl_enter();
+  pdl_wait();
+  const long long at = (long long)blockIdx.x * width;
+  float ss = 0.f;
+  if (kChunks > 0) {
+    float f[kChunks > 0 ? kChunks : 1][4], old[kChunks > 0 ? kChunks : 1][4];
+#pragma unroll
+    for (int c = 0; c < kChunks; ++c) {
+      const int col = (c * kRowThreads + threadIdx.x) * 4;
+      if (col < width) {
+        ld_elem4(y + at + col, f[c]);
+        ld_fresh4(x + at + col, old[c]);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) ss = fmaf(f[c][i], f[c][i], ss);
+      }
+    }
+    const float inv = 1.0f / sqrtf(row_sum(ss) / (float)width + eps);
+#pragma unroll
+    for (int c = 0; c < kChunks; ++c) {
+      const int col = (c * kRowThreads + threadIdx.x) * 4;
+      if (col < width) {
+        float w[4];
+        ld_elem4(weight + col, w);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) f[c][i] = fmaf(mult, f[c][i] * inv * w[i], old[c][i]);
+        st_elem4(x + at + col, f[c]);
+        if (xb) st_elem4(xb + at + col, f[c]);
+      }
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += kRowThreads) {
+      const float f = ld_elem(y + at + c);
+      ss = fmaf(f, f, ss);
+    }
+    const float inv = 1.0f / sqrtf(row_sum(ss) / (float)width + eps);
+    for (int c = threadIdx.x; c < width; c += kRowThreads) {
+      const float f = fmaf(mult, ld_elem(y + at + c) * inv * weight[c], ld_fresh(x + at + c));
+      x[at + c] = f;
+      if (xb) st_elem(xb + at + c, f);
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kRowThreads)
+silu_mul_rows_kernel(const T* __restrict__ gu, long long stride, T* __restrict__ out, long long out_stride, int rows, int ff, int vec) {
+  pdl_enter();
+  pdl_wait();
+  const int per = vec ? ff / 4 : ff;
+  const long long i = (long long)blockIdx.x * kRowThreads + threadIdx.x;
+  if (i >= (long long)rows * per) return;
+  const int r = (int)(i / per), c = (int)(i - (long long)r * per);
+  const T* src = gu + r * stride;
+  if (vec) {
+    float g[4], u[4];
+    ld_elem4(src + 4 * c, g);
+    ld_elem4(src + ff + 4 * c, u);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) g[e] = silu_f(g[e]) * u[e];
+    st_elem4(out + r * out_stride + 4 * c, g);
+  } else {
+    st_elem(out + r * out_stride + c, silu_f(ld_elem(src + c)) * ld_elem(src + ff + c));
+  }
+}
+
+// Norm of every part of a row by itself, with a gate before or after: kThreads threads per part (a warp or the block),
+// kKeep channels of it in registers per thread (0: read twice).
+template <typename T, int kThreads, int kKeep>
+__global__ void __launch_bounds__(kRowThreads)
+gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long gate_stride, int gate_first,
+                  const float* __restrict__ weight, int weight_len, float eps, float out_scale, T* __restrict__ out, long long out_stride,
+                  int rows, int len, int parts) {
+  pdl_enter();
+  const int part = len / parts;
+  const long long item = (long long)blockIdx.x * (kRowThreads / kThreads) + threadIdx.x / kThreads;
+  const int t = threadIdx.x % kThreads;
+  pdl_wait();
+  const int r = (int)(item / parts), p = (int)(item - (long long)r * parts);
+  const bool live = r < rows;  // the same for all threads of a part
+  const float* src = o + (long long)r * len + p * part;
+  const T* g = gate + r * gate_stride + p * part;
+  T* dst = out + r * out_stride + p * part;
+  auto value = [&](int c) { return gate_first ? src[c] * silu_f(ld_elem(g + c)) : src[c]; };
+  float keep[kKeep > 0 ? kKeep : 1], ss = 0.f;
+  if (live) {
+    if (kKeep > 0) {
+#pragma unroll
+      for (int i = 0; i < kKeep; ++i) {
+        const int c = t + i * kThreads;
+        keep[i] = c < part ? value(c) : 0.f;
+        ss = fmaf(keep[i], keep[i], ss);
+      }
+    } else {
+      for (int c = t; c < part; c += kThreads) {
+        const float v = value(c);
+        ss = fmaf(v, v, ss);
+      }
+    }
+  }
+  ss = kThreads == 32 ? warp_sum(ss) : row_sum(ss);
+  if (!live) return;
+  const float inv = 1.0f / sqrtf(ss / (float)part + eps);
+  auto put = [&](int c, float v) {
+    const int at = p * part + c;
+    v = v * inv * weight[weight_len == len ? at : at % weight_len] * out_scale;
+    st_elem(dst + c, gate_first ? v : v * sigmoid_f(ld_elem(g + c)));
+  };
+  if (kKeep > 0) {
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i)
+      if (t + i * kThreads < part) put(t + i * kThreads, keep[i]);
+  } else {
+    for (int c = t; c < part; c += kThreads) put(c, value(c));
+  }
+}
+
+template <typename T>
+static int run_norm_add(float* x, const void* y, const float* weight, float mult, float eps, void* xb, int rows, int width, cudaStream_t s) {
+  auto* kernel = width % 4 ? norm_add_kernel<T, 0>
+                 : width <= kRowThreads * 8 ? norm_add_kernel<T, 2>
+                 : width <= kRowThreads * 4 * kRowChunks ? norm_add_kernel<T, kRowChunks> : norm_add_kernel<T, 0>;
+  return launch_result(launch_chained(kernel, dim3(rows), dim3(kRowThreads), 0, s, x, (const T*)y, weight, mult, eps, (T*)xb, width));
+}
+
+template <typename T>
+static int run_gated_norm(const float* o, const void* gate, int64_t gate_stride, int gate_first, const float* weight, int weight_len,
+                          float eps, float out_scale, void* out, int64_t out_stride, int rows, int len, int parts,
+                          cudaStream_t s) {
+  const int part = len / parts;
+  const bool warp = part <= 32 * 8;
+  auto* kernel = part <= 128 ? gated_norm_kernel<T, 32, 4> : warp ? gated_norm_kernel<T, 32, 8>
+                 : part <= kRowThreads * 8 ? gated_norm_kernel<T, kRowThreads, 8>
+                 : part <= kRowThreads * 16 ? gated_norm_kernel<T, kRowThreads, 16> : gated_norm_kernel<T, kRowThreads, 0>;
+  const long long items = (long long)rows * parts, per = warp ? kRowThreads / 32 : 1, blocks = (items + per - 1) / per;
+  if (blocks > 0x7FFFFFF0ll) return B200KV_E_RANGE;
+  return launch_result(launch_chained(kernel, dim3((unsigned)blocks), dim3(kRowThreads), 0, s, o, (const T*)gate, (long long)gate_stride,
+                                      gate_first, weight, weight_len, eps, out_scale, (T*)out, (long long)out_stride, rows, len, parts));
+}
+
 template <typename T>
 static int run_scaled_add_norm(const float* x, const void* delta, const int32_t* index, int top, const float* weight, float alpha,
                                float eps, float* x_out, void* xb_out, int rows, int width, int32_t* zero, int num_zero,
@@ -172,4 +317,45 @@ extern "C" int b200dec_scaled_add_norm(const float* x, const void* delta, const 
   if (elem == 2)
     return run_scaled_add_norm<uint16_t>(x, delta, index, top, weight, alpha, eps, x_out, xb_out, num_rows, width, zero, num_zero, s);
   return run_scaled_add_norm<float>(x, delta, index, top, weight, alpha, eps, x_out, xb_out, num_rows, width, zero, num_zero, s);
+}
+
+extern "C" int b200dec_norm_add(float* x, const void* y, int32_t elem, const float* weight, float mult, float eps, void* xb,
+                                int32_t num_rows, int32_t width, void* stream) {
+  if (num_rows == 0) return B200KV_OK;
+  if (!x || !y || !weight) return B200KV_E_NULL;
+  if (num_rows < 0 || width < 1 || (elem != 2 && elem != 4)) return B200KV_E_SHAPE;
+  if (!aligned(x, 16) || !aligned(y, 16) || !aligned(weight, 16) || !aligned(xb, 16)) return B200KV_E_ALIGN;
+  cudaStream_t s = (cudaStream_t)stream;
+  return elem == 2 ? run_norm_add<uint16_t>(x, y, weight, mult, eps, xb, num_rows, width, s)
+                   : run_norm_add<float>(x, y, weight, mult, eps, xb, num_rows, width, s);
+}
+
+extern "C" int b200dec_silu_mul(const void* gate_up, int64_t stride, int32_t elem, void* out, int64_t out_stride, int32_t num_rows,
+                                int32_t ff, void* stream) {
+  if (num_rows == 0) return B200KV_OK;
+  if (!gate_up || !out) return B200KV_E_NULL;
+  if (num_rows < 0 || ff < 1 || stride < 2 * (int64_t)ff || out_stride < ff || (elem != 2 && elem != 4)) return B200KV_E_SHAPE;
+  const int vec = ff % 4 == 0 && stride % 4 == 0 && out_stride % 4 == 0 && aligned(gate_up, 16) && aligned(out, 16);
+  const long long items = (long long)num_rows * (vec ? ff / 4 : ff), blocks = (items + kRowThreads - 1) / kRowThreads;
+  if (blocks > 0x7FFFFFF0ll) return B200KV_E_RANGE;
+  cudaStream_t s = (cudaStream_t)stream;
+  if (elem == 2)
+    return launch_result(launch_chained(silu_mul_rows_kernel<uint16_t>, dim3((unsigned)blocks), dim3(kRowThreads), 0, s,
+                                        (const uint16_t*)gate_up, (long long)stride, (uint16_t*)out, (long long)out_stride, num_rows, ff, vec));
+  return launch_result(launch_chained(silu_mul_rows_kernel<float>, dim3((unsigned)blocks), dim3(kRowThreads), 0, s, (const float*)gate_up,
+                                      (long long)stride, (float*)out, (long long)out_stride, num_rows, ff, vec));
+}
+
+extern "C" int b200dec_gated_norm(const float* o, const void* gate, int64_t gate_stride, int32_t gate_first, int32_t elem,
+                                  const float* weight, int32_t weight_len, float eps, float out_scale, void* out, int64_t out_stride,
+                                  int32_t num_rows, int32_t len, int32_t parts, void* stream) {
+  if (num_rows == 0) return B200KV_OK;
+  if (!o || !gate || !weight || !out) return B200KV_E_NULL;
+  if (num_rows < 0 || len < 1 || parts < 1 || len % parts || weight_len < 1 || len % weight_len || (elem != 2 && elem != 4))
+    return B200KV_E_SHAPE;
+  cudaStream_t s = (cudaStream_t)stream;
+  return elem == 2 ? run_gated_norm<uint16_t>(o, gate, gate_stride, gate_first, weight, weight_len, eps, out_scale, out, out_stride,
+                                              num_rows, len, parts, s)
+                   : run_gated_norm<float>(o, gate, gate_stride, gate_first, weight, weight_len, eps, out_scale, out, out_stride, num_rows,
+                                           len, parts, s);
 }

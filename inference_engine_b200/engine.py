@@ -20,6 +20,10 @@ demand (append on decode, release on finish); a request is admitted only if the 
 need are still uncommitted, so a running request can never run out.  The first pages of the pool are a
 scratch run no request owns: padded entries of a graph replay write there.
 
+A model whose layers carry a state from token to token (`stateful`) also gets one state slot per request: taken when the
+request is admitted, given back when it ends, and never cleared, since a request at position 0 starts from zero.  Padded
+entries have slot -1, which the recurrent kernels pass over.
+
 `Scheduler` is host-only (no torch, no GPU) so that the policy is testable on its own; `Engine` adds the
 device side.  It drives any model of the registry (models/__init__.py): the model makes its own caches and runs one
 step; sampling is the library's Gumbel-max sampler (greedy at tau = 0).  Besides generating (`submit_request`, `step`),
@@ -40,6 +44,7 @@ class Request:
     prompt_ids: list[int]
     max_new_tokens: int
     pages: list[int] = field(default_factory=list)  # physical pages, in token order
+    slot: int = -1  # state slot, for models that carry a state
     committed: int = 0  # pages promised to this request at admission and not yet handed out
     cached_len: int = 0  # tokens currently in the cache
     output: list[int] = field(default_factory=list)
@@ -82,6 +87,24 @@ class PagePool:
         self.free.extend(sorted(pages, reverse=True))
 
 
+class SlotPool:
+    """State slots 0 .. n - 1, the lowest free one first."""
+
+    def __init__(self, n: int):
+        self.free = list(range(n - 1, -1, -1))
+        self.capacity = n
+
+    def take(self) -> int:
+        if not self.free:
+            raise RuntimeError("every state slot is in use")
+        return self.free.pop()
+
+    def release(self, slot: int) -> None:
+        if slot >= 0:
+            self.free.append(slot)
+            self.free.sort(reverse=True)
+
+
 @dataclass
 class Step:
     entries: list[tuple[Request, list[int]]]  # decoding requests first (one token each), then prefill chunks
@@ -98,12 +121,12 @@ class Step:
 
 class Scheduler:
     def __init__(self, max_batch_size: int, max_len: int, page_size: int, pool: PagePool, max_tokens_per_step: int,
-                 min_first_chunk: int, stop_token_id: int):
+                 min_first_chunk: int, stop_token_id: int, slots: SlotPool | None = None):
         assert max_tokens_per_step >= max_batch_size + min_first_chunk, \
             "the budget must fit every decoding request plus one first chunk, or prefill can stall forever"
         self.max_batch_size, self.max_len, self.page_size = max_batch_size, max_len, page_size
         self.pool, self.max_tokens_per_step, self.min_first_chunk = pool, max_tokens_per_step, min_first_chunk
-        self.stop_token_id = stop_token_id
+        self.stop_token_id, self.slots = stop_token_id, slots
         self.running: list[Request] = []
         self.waiting: deque[Request] = deque()
         self.next_id = 0
@@ -141,6 +164,8 @@ class Scheduler:
                 budget -= n
         while self.waiting and len(self.running) < self.max_batch_size and budget > 0:
             r = self.waiting[0]
+            if self.slots is not None and not self.slots.free:
+                break
             n = min(len(r.prompt_ids), budget)
             if n < min(len(r.prompt_ids), self.min_first_chunk):
                 break  # first come first served: nobody overtakes it
@@ -148,6 +173,8 @@ class Scheduler:
                 break  # the pool cannot promise its whole lifetime yet
             self.waiting.popleft()
             r.committed, r.admitted = self.lifetime_pages(r), True
+            if self.slots is not None:
+                r.slot = self.slots.take()
             self.running.append(r)
             entries.append((r, r.prompt_ids[:n]))
             budget -= n
@@ -172,6 +199,9 @@ class Scheduler:
                 if tok == self.stop_token_id or len(r.output) >= r.max_new_tokens or r.cached_len + 1 >= self.max_len:
                     self.pool.release(r.pages, r.committed)
                     r.pages, r.committed = [], 0
+                    if self.slots is not None:
+                        self.slots.release(r.slot)
+                        r.slot = -1
                     self.running.remove(r)
                     r.t_finish = now
                     finished.append(r)
@@ -179,11 +209,15 @@ class Scheduler:
 
 
 class Engine:
-    """Scheduler + device execution.  `model`: an instance of a registered model class on a CUDA device."""
+    """Scheduler + device execution.  `model`: an instance of a registered model class on a CUDA device.  `num_slots`: state
+    slots of a stateful model, one per live request (default: one per request of the largest batch)."""
+
+    slots: SlotPool | None = None
 
     def __init__(self, model, max_batch_size: int, max_len: int, stop_token_id: int, page_size: int | None = None,
                  num_pages: int | None = None, max_tokens_per_step: int = 1024, min_first_chunk: int = 64,
-                 max_graph_tokens: int = 512, use_graphs: bool = True, block_m: int = 128, tau: float = 0.0, seed: int = 0):
+                 max_graph_tokens: int = 512, use_graphs: bool = True, block_m: int = 128, tau: float = 0.0, seed: int = 0,
+                 num_slots: int | None = None):
         import numpy as np
         import torch
 
@@ -209,9 +243,12 @@ class Engine:
         if num_pages is None:  # what the reference's slot rows hold: max_len tokens per request
             num_pages = self.scratch_pages + max_batch_size * self.max_pages
         self.pool = PagePool(num_pages, first=self.scratch_pages)
+        if getattr(model, "stateful", False):
+            self.slots = SlotPool(max_batch_size if num_slots is None else num_slots)
         self.sched = Scheduler(max_batch_size, max_len, page_size, self.pool, max_tokens_per_step, min_first_chunk,
-                               stop_token_id)
-        self.caches = model.make_caches(num_pages, page_size, self.max_pages * page_size)
+                               stop_token_id, self.slots)
+        per_slot = {} if self.slots is None else {"slots": self.slots.capacity}
+        self.caches = model.make_caches(num_pages, page_size, self.max_pages * page_size, **per_slot)
         # one int32 buffer per kind of step, filled on the host and copied in one piece
         cap = sum(self.mixed_layout(max_tokens_per_step))
         self.host_mixed = torch.empty(cap, dtype=torch.int32).pin_memory()
@@ -282,6 +319,8 @@ class Engine:
             if not self.pool.commit(need):
                 raise RuntimeError("the page pool is exhausted")
             r.pages.extend(self.pool.take() for _ in range(need))
+            if self.slots is not None and r.slot < 0:
+                r.slot = self.slots.take()
         step = Step([entries[i][:2] for i in order], decoding)
         out = self.run(step)
         first, at = {}, 0
@@ -299,21 +338,24 @@ class Engine:
     def close_replay(self, r: Request) -> None:
         self.pool.release(r.pages)
         r.pages = []
+        if self.slots is not None:
+            self.slots.release(r.slot)
+            r.slot = -1
         self.rows.pop(r.id, None)
 
     # ------------------------------------------------------------------ input buffers
     def mixed_layout(self, n_tokens: int) -> list[int]:
         """Field lengths of a step with prefill padded to n_tokens: ids, positions, seq_ids, cu_seqlens,
-        cached_lens, cu_cached, tile_start, num_decoding, block table.  The same n_tokens always gives the
+        cached_lens, cu_cached, tile_start, num_decoding, block table, state slots.  The same n_tokens always gives the
         same layout, so a bucket's fields always sit at the same addresses."""
         E = self.num_entries
-        return [n_tokens, n_tokens, n_tokens, E + 1, E, E + 1, math.ceil(n_tokens / self.block_m) + E, 1, E * self.max_pages]
+        return [n_tokens, n_tokens, n_tokens, E + 1, E, E + 1, math.ceil(n_tokens / self.block_m) + E, 1, E * self.max_pages, E]
 
     def decode_layout(self) -> list[int]:
-        """ids, cached_lens, num_decoding, block table of a pure-decode step, sized for the largest batch; a
+        """ids, cached_lens, num_decoding, block table, state slots of a pure-decode step, sized for the largest batch; a
         bucket of b rows uses the first b of each (same start addresses for every bucket)."""
         B = self.max_batch_size
-        return [B, B, 1, B * self.max_pages]
+        return [B, B, 1, B * self.max_pages, B]
 
     def table_row(self, r: Request):
         """The request's block-table row as an int32 array, extended in place as pages are appended."""
@@ -346,6 +388,9 @@ class Engine:
             table[i] = self.table_row(r)
         table[len(step.entries)] = self.scratch_row  # the padding entry lives on the scratch run
         table[len(step.entries) + 1 :] = 0
+        slots = buf[offs[9] : offs[10]]
+        slots[:] = -1
+        slots[: len(step.entries)] = [r.slot for r, _ in step.entries]
         self.dev_mixed[: len(buf)].copy_(self.host_mixed[: len(buf)], non_blocking=True)
         return plan["cu_cached"][-1]
 
@@ -354,7 +399,7 @@ class Engine:
         v = self.dev_mixed[: sum(self.mixed_layout(n_pad))].split(self.mixed_layout(n_pad))
         inp = S.StepInputs(ids=v[0], positions=v[1], seq_ids=v[2], cu_seqlens=v[3], cached_lens=v[4], cu_cached=v[5],
                            tile_start=v[6], num_decoding=v[7], block_table=v[8].view(self.num_entries, self.max_pages),
-                           prefix_tokens=prefix_tokens, block_m=self.block_m)
+                           prefix_tokens=prefix_tokens, block_m=self.block_m, slots=v[9])
         if self.prefix is None:
             return inp, None
         # a step whose cached prefixes exceed the scratch gets a one-off buffer
@@ -363,17 +408,19 @@ class Engine:
 
     def decode_views(self, b: int):
         B = self.max_batch_size
-        ids, cached, nd, table = self.dev_decode.split(self.decode_layout())
-        return ids[:b], cached[:b], nd, table.view(B, self.max_pages)[:b]
+        ids, cached, nd, table, slots = self.dev_decode.split(self.decode_layout())
+        return ids[:b], cached[:b], nd, table.view(B, self.max_pages)[:b], slots[:b]
 
     # ------------------------------------------------------------------ execution
     def forward_mixed(self, n_pad: int, prefix_tokens: int = 0):
         inp, prefix = self.mixed_views(n_pad, prefix_tokens)
-        return self.model.step(self.caches, inp, inp.ids, inp.cached_lens, inp.block_table, inp.num_decoding, prefix)
+        state = {} if self.slots is None else {"slots": inp.slots}
+        return self.model.step(self.caches, inp, inp.ids, inp.cached_lens, inp.block_table, inp.num_decoding, prefix, **state)
 
     def forward_decode(self, b: int):
-        ids, cached, nd, table = self.decode_views(b)
-        return self.model.step(self.caches, None, ids, cached, table, nd)
+        ids, cached, nd, table, slots = self.decode_views(b)
+        state = {} if self.slots is None else {"slots": slots}
+        return self.model.step(self.caches, None, ids, cached, table, nd, **state)
 
     def capture_graph(self, run):
         """Two eager runs first (engine.py:432-449), then the recording; returns (graph, the step's output)."""
@@ -394,7 +441,7 @@ class Engine:
         on the device) and one per token bucket (any mix of entries that fits, engine.py:412-430).  The dummy
         inputs during capture are a single padding entry on the scratch run, so what the warm-up writes is
         harmless."""
-        self.dev_decode.zero_()
+        self.dev_decode.zero_()  # nothing decodes
         for b in reversed(self.graph_buckets):
             self.decode_graphs[b] = self.capture_graph(lambda b=b: self.forward_decode(b))
         for n in reversed(self.token_buckets):
@@ -421,10 +468,12 @@ class Engine:
         buf[B:Bm] = 0
         buf[Bm + B : 2 * Bm] = 0
         buf[2 * Bm] = B
-        table = buf[2 * Bm + 1 :].reshape(Bm, self.max_pages)
+        table = buf[2 * Bm + 1 : -Bm].reshape(Bm, self.max_pages)
         for i, (r, _) in enumerate(step.entries):
             table[i] = self.table_row(r)
         table[B:] = 0
+        buf[-Bm:] = -1
+        buf[len(buf) - Bm : len(buf) - Bm + B] = [r.slot for r, _ in step.entries]
         self.dev_decode.copy_(self.host_decode, non_blocking=True)
         self.seconds["inputs"] += time.perf_counter() - t_in
         if b in self.decode_graphs:

@@ -8,6 +8,8 @@ and its instances what the engine drives:
     make_prefix(max_len) / None                    scratch for the prefilling entries' cached tokens, if it wants one
     step(caches, inp, ids, cached_lens, block_table, num_decoding, prefix) -> StepOutput
     logits(hidden)                                 fp32 or bf16 logits of normed rows
+A class with `stateful = True` keeps a state per request beside the pages: its make_caches takes slots=, the number of state
+slots, and its step slots=, int32 [entries], the slot of every entry (-1: padding).
 """
 from __future__ import annotations
 
@@ -35,7 +37,7 @@ def register(architecture: str):
 def load_all() -> dict[str, type]:
     """Import every model module (each registers itself)."""
     from .. import scaffold  # noqa: F401  (registers itself)
-    from . import radivik  # noqa: F401
+    from . import biranex, radivik  # noqa: F401
 
     return MODELS
 

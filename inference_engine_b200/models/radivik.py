@@ -16,6 +16,7 @@ import torch
 
 from .. import kernels as K
 from .. import ops
+from ..checkpoint import RandomWeights
 from . import StepOutput, register
 
 GATE_SLOPE = 1.702  # y = g * sigmoid(slope * g) * (u + 1)
@@ -196,14 +197,3 @@ class Radivik:
 
     def logits(self, hidden: torch.Tensor) -> torch.Tensor:
         return K.linear(hidden, self.head, out_dtype=torch.float32)
-
-
-class RandomWeights:
-    """Stand-in for a checkpoint: matrices ~ N(0, 1 / fan-in), norms near 1, drawn on the device."""
-
-    def __init__(self, device, seed: int = 0):
-        self.device, self.g = device, torch.Generator(device=device).manual_seed(seed)
-
-    def take(self, name: str, *shape: int) -> torch.Tensor:
-        t = torch.randn(*shape, generator=self.g, device=self.device)
-        return (1.0 + 0.1 * t if len(shape) == 1 else t * shape[-1] ** -0.5).to(torch.bfloat16)

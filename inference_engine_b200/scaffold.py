@@ -61,6 +61,7 @@ class StepInputs:
     block_table: torch.Tensor  # int32 [S, max_pages]
     prefix_tokens: int
     block_m: int
+    slots: torch.Tensor | None = None  # int32 [S]: state slots, for models that carry a state
 
 
 def plan_step(
