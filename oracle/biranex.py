@@ -151,16 +151,17 @@ def dense(h, w, p):
     return (silu(h @ w[p + "gate"].T) * (h @ w[p + "up"].T)) @ w[p + "down"].T
 
 
-def forward(cfg, weights, tokens, dtype=np.float64):
-    """(logits [T, vocab], residual after every layer [layers, T, width])."""
+def forward(cfg, weights, tokens, dtype=np.float64, read=lambda x: x):
+    """(logits [T, vocab], residual after every layer [layers, T, width]).  `read`: what a sublayer sees of the residual, for
+    estimates of what rounding alone does."""
     w = {n: np.asarray(a, dtype) for n, a in weights.items()}
     eps, mult = cfg["norm"]["eps"], cfg["residual_mult"]
     x, trace = w["embed"][np.asarray(tokens)], []
     for i, layer in enumerate(cfg["layers"]):
         p = f"l{i}."
         mixer = {"parallel": parallel, "channel_delta": channel_delta}[layer["type"]]
-        x = x + mult * rms_norm(mixer(x, w, p + "mix.", layer["mixer"], eps), eps, w[p + "norm1"])
+        x = x + mult * rms_norm(mixer(read(x), w, p + "mix.", layer["mixer"], eps), eps, w[p + "norm1"])
         if layer["mlp"]:
-            x = x + mult * rms_norm(dense(x, w, p + "mlp."), eps, w[p + "norm2"])
+            x = x + mult * rms_norm(dense(read(x), w, p + "mlp."), eps, w[p + "norm2"])
         trace.append(x)
-    return rms_norm(x, eps, w["final.norm"]) @ w["embed"].T, np.stack(trace)
+    return read(rms_norm(x, eps, w["final.norm"])) @ w["embed"].T, np.stack(trace)
