@@ -15,6 +15,7 @@ rank's device time.  Prints ONE JSON line on rank 0.
 from __future__ import annotations
 
 import argparse
+import ctypes
 import json
 import math
 import os
@@ -881,12 +882,76 @@ def run_prefill(args):
         print(json.dumps({"case": "prefill_attention", "prior_context": prior, "max_abs_diff_between_kernels": diff}), flush=True)
 
 
+class RooflineBench:
+    """Kernels against their rooflines: algorithmic bytes over the measured copy bandwidth or FLOPs over the measured bf16
+    GEMM rate, whichever takes longer; calls captured in one CUDA graph over as many distinct inputs as exceed L2, median of
+    `steps` replays."""
+
+    L2 = 160e6
+
+    def __init__(self, args, seed: int):
+        import torch
+
+        from inference_engine_b200 import kernels as K
+
+        self.torch, self.K, self.args = torch, K, args
+        self.dev = torch.device("cuda", 0)
+        torch.cuda.set_device(self.dev)
+        K.set_early_start(not args.no_early_start)
+        self.hbm = peaks()[0] * 1e9
+        tf = 1590.0
+        if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
+            with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
+                tf = float(json.load(f)["bf16_tflops"])
+        self.tf = tf * 1e12
+        self.gen = torch.Generator(device=self.dev).manual_seed(seed)
+
+    def rnd(self, *shape, dtype=None):
+        return self.torch.randn(*shape, generator=self.gen, device=self.dev).to(dtype or self.torch.bfloat16)
+
+    def i32(self, x):
+        return self.torch.tensor(x, dtype=self.torch.int32, device=self.dev)
+
+    def graph_us(self, calls):
+        torch = self.torch
+        with torch.inference_mode():
+            for _ in range(2):
+                for c in calls:
+                    c()
+            torch.cuda.synchronize()
+            g = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(g):
+                for c in calls:
+                    c()
+        for _ in range(max(self.args.warmup, 3)):
+            g.replay()
+        torch.cuda.synchronize()
+        ts = []
+        for _ in range(self.args.steps):
+            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            e0.record()
+            g.replay()
+            e1.record()
+            torch.cuda.synchronize()
+            ts.append(e0.elapsed_time(e1) * 1e3 / len(calls))
+        return statistics.median(ts)
+
+    def report(self, group, model, kernel, calls, nbytes, flops=0.0, peak=None):
+        """peak: another rate than the bf16 one the FLOPs are held against (the 32-bit rate of the CUDA cores)."""
+        us = self.graph_us(calls)
+        roof = max(nbytes / self.hbm, flops / (peak or self.tf)) * 1e6
+        print(json.dumps({"group": group, "model": model, "kernel": kernel, "us": round(us, 2), "roofline_us": round(roof, 2),
+                          "of_roofline": round(roof / us, 3), "gbs": round(nbytes / us / 1e3), "tflops": round(flops / us / 1e6, 1),
+                          "status": self.K.check_status(self.dev)}), flush=True)
+
+    def sets(self, nbytes):
+        return max(2, min(24, math.ceil(self.L2 / nbytes)))
+
+
 def run_radivik(args):
     """--radivik: the Radivik decoder beside the DecoderScaffold at equal size (random weights).
 
-    (1) every kernel of the new design and the like kernel of the scaffold, as fractions of their rooflines: algorithmic
-    bytes over the measured copy bandwidth or FLOPs over the measured bf16 GEMM rate, whichever takes longer; calls
-    captured in one CUDA graph over as many distinct inputs as exceed L2, median of `steps` replays;
+    (1) every kernel of the new design and the like kernel of the scaffold, as fractions of their rooflines (RooflineBench);
     (2) model steps through the registry's classes: a 1024-token prompt portion on 3072 cached tokens, and a pure decode
     step of 64 entries with 4096 tokens each."""
     import torch
@@ -897,57 +962,8 @@ def run_radivik(args):
     from inference_engine_b200.models import model_class
     from inference_engine_b200.models.radivik import GATE_SLOPE
 
-    dev = torch.device("cuda", 0)
-    torch.cuda.set_device(dev)
-    K.set_early_start(not args.no_early_start)
-    hbm = peaks()[0] * 1e9
-    tf = 1590.0
-    if os.path.exists(os.path.join(ROOT, "MEASURED_PEAKS.json")):
-        with open(os.path.join(ROOT, "MEASURED_PEAKS.json")) as f:
-            tf = float(json.load(f)["bf16_tflops"])
-    tf *= 1e12
-    L2 = 160e6
-    gen = torch.Generator(device=dev).manual_seed(6)
-
-    def rnd(*shape, dtype=torch.bfloat16):
-        return torch.randn(*shape, generator=gen, device=dev).to(dtype)
-
-    def i32(x):
-        return torch.tensor(x, dtype=torch.int32, device=dev)
-
-    def graph_us(calls):
-        with torch.inference_mode():
-            for _ in range(2):
-                for c in calls:
-                    c()
-            torch.cuda.synchronize()
-            g = torch.cuda.CUDAGraph()
-            with torch.cuda.graph(g):
-                for c in calls:
-                    c()
-        for _ in range(max(args.warmup, 3)):
-            g.replay()
-        torch.cuda.synchronize()
-        ts = []
-        for _ in range(args.steps):
-            e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-            e0.record()
-            g.replay()
-            e1.record()
-            torch.cuda.synchronize()
-            ts.append(e0.elapsed_time(e1) * 1e3 / len(calls))
-        return statistics.median(ts)
-
-    def report(group, model, kernel, calls, nbytes, flops=0.0):
-        us = graph_us(calls)
-        roof = max(nbytes / hbm, flops / tf) * 1e6
-        print(json.dumps({"group": group, "model": model, "kernel": kernel, "us": round(us, 2), "roofline_us": round(roof, 2),
-                          "of_roofline": round(roof / us, 3), "gbs": round(nbytes / us / 1e3), "tflops": round(flops / us / 1e6, 1),
-                          "status": K.check_status(dev)}), flush=True)
-
-    def sets(nbytes):
-        return max(2, min(24, math.ceil(L2 / nbytes)))
-
+    b = RooflineBench(args, seed=6)
+    dev, gen, hbm, tf, rnd, i32, graph_us, report, sets = b.dev, b.gen, b.hbm, b.tf, b.rnd, b.i32, b.graph_us, b.report, b.sets
     W, FF = S.HIDDEN, S.FFN
     sizes = {  # name: heads, kv heads, key size, value size, rotated channels, experts, top, ff
         "as the scaffold": (16, 8, 128, 128, 128, 8, 2, FF // 2),
@@ -1172,6 +1188,235 @@ def run_radivik(args):
             mlp_case(N)
         model_case()
     print(json.dumps({"clocks": clk.summary(), "hbm_gbs": hbm / 1e9, "bf16_tflops": tf / 1e12, "data": "random weights and inputs"}), flush=True)
+
+
+def run_biranex(args):
+    """--biranex: the Biranex decoder beside Radivik and the DecoderScaffold at equal size (random weights).
+
+    (1) every kernel of the new design and the like kernel of the other two, as fractions of their rooflines (RooflineBench).
+    Attention counts visible (query, key) pairs.  The state recurrences count their 32-bit multiply-adds against the CUDA
+    cores' 32-bit rate (SMs x 128 lanes x 2 x 1.965 GHz) and their bytes, whichever takes longer; they have no like kernel, so a
+    bandwidth-bound neighbour stands beside them;
+    (2) model steps through the registry's classes: a 1024-token prompt portion on 3072 cached tokens, the same as the first
+    portion of a prompt, and a pure decode step of 64 entries with 4096 tokens each."""
+    import torch
+
+    from inference_engine_b200 import kernels as K
+    from inference_engine_b200 import ops
+    from inference_engine_b200 import scaffold as S
+    from inference_engine_b200.models import model_class
+
+    b = RooflineBench(args, seed=7)
+    dev, gen, rnd, i32, report, sets = b.dev, b.gen, b.rnd, b.i32, b.report, b.sets
+    fp32 = K.num_sms(dev) * 128 * 2 * 1.965e9
+    bf16, W, FF, PG = torch.bfloat16, S.HIDDEN, S.FFN, 64
+    sizes = {  # left (heads, kv, dim, vdim, window, rotated), right (heads, groups, state, vdim), delta (heads, kv, dim, vdim)
+        "A": ((16, 8, 128, 128, 1024, 128), (64, 8, 128, 64), (16, 16, 128, 128)),
+        "B": ((32, 8, 64, 64, 512, 32), (48, 1, 64, 64), (12, 6, 96, 112)),
+    }
+
+    def parallel(sz):
+        (h, kv, d, vd, win, rot), (sh, g, n, p), _ = sz
+        return {"type": "parallel", "mlp": {"kind": "dense", "ff": FF}, "mixer": {
+            "left_scale": 1.0, "right_scale": 1.0,
+            "left": {"heads": h, "kv_heads": kv, "dim": d, "vdim": vd, "scale": d ** -0.5, "mask": {"size": win},
+                     "rot": {"dims": rot, "base": 1e6, "scaling": {"factor": 2.0}}},
+            "right": {"heads": sh, "groups": g, "state": n, "vdim": p, "conv": 4, "norm_groups": g}}}
+
+    def delta(sz):
+        h, kv, d, vd = sz[2]
+        return {"type": "channel_delta", "mlp": {"kind": "dense", "ff": FF},
+                "mixer": {"heads": h, "kv_heads": kv, "dim": d, "vdim": vd, "conv": 4}}
+
+    def config(layers, vocab):
+        return {"architecture": "Biranex", "vocab": vocab, "width": W, "residual_mult": 0.5, "norm": {"eps": 1e-6}, "layers": layers}
+
+    def prompt_rows(chunks, prior):
+        n, E = sum(chunks), len(chunks)
+        plan = S.plan_step([], [(prior, c) for c in chunks], n, E + 1)
+        table, pages = S.assign_pages(plan, PG, (prior + max(chunks)) // PG + 1)
+        inp = S.upload_step(plan, table, [0] * n, dev)
+        rows = ops.Rows(n, inp.cached_lens, inp.num_decoding, inp.block_table, inp.seq_ids, inp.positions, inp.cu_seqlens, inp.tile_start, 128)
+        rows.slots = i32(list(range(E)) + [-1])
+        return rows, pages, inp
+
+    # ------------------------------------------------------------------ attention
+    def attention_cases():
+        for prior, chunk in ((3072, 992), (0, 992)):
+            group = f"prompt attention, {chunk} rows on {prior}"
+            rows, pages, _ = prompt_rows([chunk], prior)
+            for name, (left, _, _) in sizes.items():
+                h, kv, d, vd, win, _ = left
+                nb = (prior + chunk) * kv * (d + vd) * 2
+                caches = [ops.make_paged_kv(pages, kv, PG, d, vd, bf16, dev) for _ in range(sets(nb))]
+                for c in caches:
+                    c.k.normal_(generator=gen)
+                    c.v.normal_(generator=gen)
+                q, out, sink, gate = rnd(chunk, h, d), torch.empty(chunk, h, vd, dtype=bf16, device=dev), torch.zeros(h, device=dev), rnd(chunk, h)
+                pos = torch.arange(prior, prior + chunk)
+                for who, w, opt in (("Radivik", 0, None), ("Biranex, window 0", 0, ops.AttnOptions(0, sink, gate)),
+                                    (f"Biranex, window {win}", win, ops.AttnOptions(win, sink, gate))):
+                    pairs = int((pos + 1 if not w else (pos + 1).clamp(max=w)).sum())
+                    seen = min(prior + chunk, chunk + w - 1) if w else prior + chunk
+                    report(group, f"{name}: {who}", "paged_prefill_attention",
+                           [lambda c=c: ops.paged_prefill_attention(q, c, rows, d ** -0.5, out, opt) for c in caches],
+                           seen * kv * (d + vd) * 2 + chunk * h * (d + vd) * 2, 2.0 * (d + vd) * pairs * h)
+                del caches
+        for B, ctx in ((64, 4096), (8, 2048)):
+            for name, (left, _, _) in sizes.items():
+                h, kv, d, vd, win, _ = left
+                group = f"decode attention, {B} entries of {ctx}"
+                P = ctx // PG
+                table = torch.randperm(B * P, generator=gen, device=dev).to(torch.int32).view(B, P)
+                rows = ops.Rows(B, i32([ctx - 1] * B), i32([B]), table)
+                short = ops.Rows(B, i32([win - 1] * B), i32([B]), table)
+                caches = [ops.make_paged_kv(B * P, kv, PG, d, vd, bf16, dev) for _ in range(sets(B * win * kv * (d + vd) * 2))]
+                for c in caches:
+                    c.k.normal_(generator=gen)
+                    c.v.normal_(generator=gen)
+                q, out, sink, gate = rnd(B, h, d), torch.empty(B, h, vd, dtype=bf16, device=dev), torch.zeros(h, device=dev), rnd(B, h)
+                for who, r, seen, opt in (("Radivik", rows, ctx, None), ("Biranex, window 0", rows, ctx, ops.AttnOptions(0, sink, gate)),
+                                          (f"Radivik, entries of {win}", short, win, None),
+                                          (f"Biranex, window {win}", rows, win, ops.AttnOptions(win, sink, gate))):
+                    report(group, f"{name}: {who}", "paged_decode_attention",
+                           [lambda c=c: ops.paged_decode_attention(q, c, r, d ** -0.5, out, True, opt) for c in caches],
+                           B * seen * kv * (d + vd) * 2 + B * h * (d + vd) * 2)
+                del caches
+
+    def write_case(N, decode):
+        group = f"norm, rotation and cache write, {N} rows" + (" (decode)" if decode else "")
+        for name, (left, _, _) in sizes.items():
+            h, kv, d, vd, _, rot = left
+            if decode:
+                P = 9
+                table = torch.randperm(N * P, generator=gen, device=dev).to(torch.int32).view(N, P)
+                rows, pages = ops.Rows(N, i32([512] * N), i32([N]), table), N * P
+            else:
+                rows, pages, _ = prompt_rows([N], 512)
+            nb = N * 2 * 2 * ((h + kv) * d + kv * vd)
+            k = sets(nb)
+            caches = [ops.make_paged_kv(pages, kv, PG, d, vd, bf16, dev) for _ in range(k)]
+            qkv = [rnd(N, (h + kv) * d + kv * vd) for _ in range(k)]
+            cs, qn, kn = ops.Rotary(rot, 1e6).table(512 + N + 1, dev), torch.ones(h * d, device=dev), torch.ones(kv * d, device=dev)
+            report(group, f"{name}: Radivik", "rope_write", [lambda t=t, c=c: ops.rope_write(t, rows, c, cs, h, True, True, 1e-6)
+                                                             for t, c in zip(qkv, caches)], nb)
+            report(group, f"{name}: Biranex", "norm_rope_write", [lambda t=t, c=c: ops.norm_rope_write(t, rows, c, qn, kn, 1e-6, cs, h)
+                                                                  for t, c in zip(qkv, caches)], nb)
+
+    # ------------------------------------------------------------------ row ops
+    def row_cases(N):
+        group = f"residual and norm, {N} rows"
+        nb, wf = N * W * 12, torch.ones(W, device=dev)
+        a = [(rnd(N, W, dtype=torch.float32), rnd(N, W)) for _ in range(sets(nb))]
+        report(group, "Radivik", "scaled_add_norm", [lambda t=t: ops.scaled_add_norm(*t, wf, 2.0, 1e-6, bf16) for t in a], nb)
+        report(group, "Biranex", "norm_add", [lambda t=t: ops.norm_add(*t, wf, 0.1, 1e-6, bf16) for t in a], nb)
+        group, nb = f"gated unit of the feed-forward, {N} rows", 2 * 3 * N * FF
+        x = [rnd(N, 2 * FF) for _ in range(sets(nb))]
+        report(group, "scaffold", "silu_mul", [lambda t=t: K.silu_mul(t) for t in x], nb)
+        report(group, "Biranex", "silu_mul", [lambda t=t: ops.silu_mul(t, FF) for t in x], nb)
+        for name, (_, (sh, g, n, p), _) in sizes.items():
+            group, L = f"gated norm of the state-space output, {N} rows", sh * p
+            nb = N * L * 8
+            a = [(rnd(N, L, dtype=torch.float32), rnd(N, L), torch.empty(N, L, dtype=bf16, device=dev)) for _ in range(sets(nb))]
+            norm = ops.GatedNorm(torch.ones(L, device=dev), g, 1e-6, True)
+            report(group, f"{name}: Biranex", "gated_norm", [lambda t=t: ops.gated_norm(t[0], t[1], norm, t[2]) for t in a], nb)
+
+    # ------------------------------------------------------------------ recurrences
+    def recurrences(sz):
+        cfg = config([parallel(sz), delta(sz)], 64)
+        m = model_class(cfg).from_config(cfg, None, dev)
+        return (("state space", m.layers[0].mixer.rec, 4), ("delta rule", m.layers[1].mixer.rec, 8))
+
+    def rec_data(rec, N, k):
+        step = rec.dt_bias.numel()
+        return [(rnd(N, rec.channels), rnd(N, step), rnd(N, rec.heads) if rec.correct else None) for _ in range(k)]
+
+    def recurrence_decode_case(B):
+        for name, sz in sizes.items():
+            for kind, rec, per in recurrences(sz):
+                nb = B * rec.heads * rec.dim * rec.vdim * 8 + B * (rec.channels * 2 * (rec.taps + 1) + rec.dt_bias.numel() * 2 + rec.heads * rec.vdim * 4)
+                k = sets(nb)
+                sts, data = [ops.make_recurrent_state(rec, B, bf16, dev) for _ in range(k)], rec_data(rec, B, k)
+                rows = ops.Rows(B, i32([777] * B), i32([B]), i32([[0]] * B), slots=torch.randperm(B, generator=gen, device=dev).to(torch.int32))
+                out = torch.empty(B, rec.heads * rec.vdim, device=dev)
+                report(f"recurrence, decode, {B} entries", f"{name}: Biranex, {kind}", "recurrence_decode",
+                       [lambda s=s, d=d: ops.recurrence_decode(rec, s, *d, rows, out) for s, d in zip(sts, data)], nb)
+                if rec.correct:
+                    norm, gate = ops.GatedNorm(torch.ones(rec.vdim, device=dev), rec.heads, 1e-6, False), rnd(B, rec.heads * rec.vdim)
+                    o16 = torch.empty(B, rec.heads * rec.vdim, dtype=bf16, device=dev)
+                    report(f"recurrence, decode, {B} entries", f"{name}: Biranex, {kind}, with the gated norm", "recurrence_decode",
+                           [lambda s=s, d=d: ops.recurrence_decode(rec, s, *d, rows, o16, norm, gate) for s, d in zip(sts, data)], nb)
+
+    def recurrence_prompt_case(chunks):
+        N, prior = sum(chunks), 512
+        for name, sz in sizes.items():
+            for kind, rec, per in recurrences(sz):
+                rows, _, _ = prompt_rows(chunks, prior)
+                nb = N * (rec.channels * 2 + rec.dt_bias.numel() * 2 + rec.heads * rec.vdim * 4)
+                k = sets(nb)
+                sts, data = [ops.make_recurrent_state(rec, len(chunks), bf16, dev) for _ in range(k)], rec_data(rec, N, k)
+                out = torch.empty(N, rec.heads * rec.vdim, device=dev)
+                group = f"recurrence, {len(chunks)} portions of {chunks[0]} tokens"
+                report(group, f"{name}: Biranex, {kind}", "convolution + scan",
+                       [lambda s=s, d=d: ops.recurrence_prefill(rec, s, *d, rows, out) for s, d in zip(sts, data)], nb,
+                       N * rec.heads * rec.dim * rec.vdim * float(per), fp32)
+                conv, lib, st = torch.empty(N, rec.channels, dtype=bf16, device=dev), ops._lib_dec(), K.status_word(dev).data_ptr()
+
+                def only_conv(s, d):
+                    r, i = ops._recurrence_args(rec, s, *d)
+                    e = rows.entries()
+                    lib.b200dec_conv_rows(ctypes.byref(r), ctypes.byref(i), ctypes.byref(e), conv.data_ptr(), st, K._stream())
+
+                report(group, f"{name}: Biranex, {kind}", "convolution alone", [lambda s=s, d=d: only_conv(s, d) for s, d in zip(sts, data)],
+                       N * rec.channels * 4)
+
+    # ------------------------------------------------------------------ whole steps
+    def model_case():
+        layers, vocab, B, ctx = 8, 32768, 64, 4096
+        rad = {"architecture": "Radivik", "vocab": vocab, "width": W, "postln_alpha": 2.0, "norm": {"eps": 1e-6}, "layers": [
+            {"type": "attention", "mixer": {"heads": 16, "kv_heads": 8, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"dims": 128, "base": 1e6}},
+             "mlp": {"kind": "moe", "expert": {"ff": FF // 2, "limit": 7.0}, "router": {"experts": 8, "top": 2}}}] * layers}
+        models = [("scaffold", {"architecture": "DecoderScaffold", "hidden": W, "ffn": FF, "vocab": vocab, "layers": layers}, PAGE), ("Radivik A", rad, PG)]
+        for name, sz in sizes.items():
+            models += [(f"Biranex {name}, parallel and delta layers in turn", config([parallel(sz), delta(sz)] * (layers // 2), vocab), PG),
+                       (f"Biranex {name}, parallel layers", config([parallel(sz)] * layers, vocab), PG),
+                       (f"Biranex {name}, delta layers", config([delta(sz)] * layers, vocab), PG)]
+        for name, cfg, page in models:
+            m = model_class(cfg).from_config(cfg, None, dev)
+            P, stateful = ctx // page, getattr(m, "stateful", False)
+            caches = m.make_caches(B * P, page, ctx, **({"slots": B} if stateful else {}))
+            for prior, chunk in ((3072, 1024), (0, 1024)):
+                plan = S.plan_step([], [(prior, chunk)], chunk, 2)
+                table = torch.zeros(2, P, dtype=torch.int32)
+                table[0] = torch.arange(P)
+                inp = S.upload_step(plan, table, torch.randint(0, vocab, (chunk,)).tolist(), dev)
+                prefix = m.make_prefix(ctx)
+                prefix = None if prefix is None else S.PrefixScratch(*prefix, inp.cu_cached)
+                state = {"slots": i32([0, -1])} if stateful else {}
+                us = b.graph_us([lambda: m.step(caches, inp, inp.ids, inp.cached_lens, inp.block_table, inp.num_decoding, prefix, **state)])
+                print(json.dumps({"case": f"prompt portion of {chunk} tokens on {prior}, {layers} layers", "model": name, "ms": round(us / 1e3, 3),
+                                  "tokens_per_s": round(chunk / us * 1e6)}), flush=True)
+            tab = torch.randperm(B * P, generator=gen, device=dev).to(torch.int32).view(B, P)
+            ids, cached, nd = i32(list(range(B))), i32([ctx - 1] * B), i32([B])
+            state = {"slots": i32(list(range(B)))} if stateful else {}
+            us = b.graph_us([lambda: m.step(caches, None, ids, cached, tab, nd, **state)])
+            print(json.dumps({"case": f"decode step of {B} entries of {ctx}, {layers} layers", "model": name, "ms": round(us / 1e3, 3),
+                              "tokens_per_s": round(B / us * 1e6), "status": K.check_status(dev)}), flush=True)
+            del caches, m
+
+    with ClockSampler(0) as clk:
+        attention_cases()
+        write_case(64, True)
+        write_case(1024, False)
+        for N in (64, 1024, 4096):
+            row_cases(N)
+        for B in (8, 64, 256):
+            recurrence_decode_case(B)
+        for chunks in ([1024], [256] * 8):
+            recurrence_prompt_case(chunks)
+        model_case()
+    print(json.dumps({"clocks": clk.summary(), "hbm_gbs": b.hbm / 1e9, "bf16_tflops": b.tf / 1e12, "fp32_tflops": fp32 / 1e12,
+                      "data": "random weights and inputs"}), flush=True)
 
 
 def run_mixed(args):
@@ -1894,9 +2139,13 @@ def main():
     ap.add_argument("--linear", action="store_true", help="weight-streaming matmul for few rows beside cuBLAS")
     ap.add_argument("--phases", action="store_true", help="per-phase and per-SM times of the decode kernel (instrumented build)")
     ap.add_argument("--radivik", action="store_true", help="the Radivik decoder beside the scaffold: kernels against their rooflines, whole steps")
+    ap.add_argument("--biranex", action="store_true", help="the Biranex decoder beside Radivik and the scaffold: kernels against their rooflines, "
+                    "whole steps")
     args = ap.parse_args()
     if args.radivik:
         run_radivik(args)
+    elif args.biranex:
+        run_biranex(args)
     elif args.phases:
         run_phases(args)
     elif args.linear:

@@ -40,6 +40,39 @@ __device__ __forceinline__ void st_elem4(uint16_t* p, const float (&f)[4]) {
   *reinterpret_cast<uint2*>(p) = v;
 }
 
+// kVec consecutive elements (aligned to their size; 8 bf16 in one 16-byte access)
+__device__ __forceinline__ void ld_vec(const uint16_t* p, float (&f)[1]) { f[0] = ld_elem(p); }
+__device__ __forceinline__ void ld_vec(const float* p, float (&f)[1]) { f[0] = *p; }
+__device__ __forceinline__ void ld_vec(const uint16_t* p, float (&f)[4]) { ld_elem4(p, f); }
+__device__ __forceinline__ void ld_vec(const float* p, float (&f)[4]) { ld_elem4(p, f); }
+__device__ __forceinline__ void unpack8(const uint4& v, float (&f)[8]) {
+  f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xFFFF0000u);
+  f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xFFFF0000u);
+  f[4] = __uint_as_float(v.z << 16); f[5] = __uint_as_float(v.z & 0xFFFF0000u);
+  f[6] = __uint_as_float(v.w << 16); f[7] = __uint_as_float(v.w & 0xFFFF0000u);
+}
+__device__ __forceinline__ void ld_vec(const uint16_t* p, float (&f)[8]) { unpack8(*reinterpret_cast<const uint4*>(p), f); }
+__device__ __forceinline__ void ld_vec(const float* p, float (&f)[8]) {
+  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+  f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+__device__ __forceinline__ void st_vec(uint16_t* p, const float (&f)[1]) { st_elem(p, f[0]); }
+__device__ __forceinline__ void st_vec(float* p, const float (&f)[1]) { *p = f[0]; }
+__device__ __forceinline__ void st_vec(uint16_t* p, const float (&f)[4]) { st_elem4(p, f); }
+__device__ __forceinline__ void st_vec(float* p, const float (&f)[4]) { st_elem4(p, f); }
+__device__ __forceinline__ void st_vec(uint16_t* p, const float (&f)[8]) {
+  uint4 v;
+  v.x = float_to_bf16_bits(f[0]) | (float_to_bf16_bits(f[1]) << 16);
+  v.y = float_to_bf16_bits(f[2]) | (float_to_bf16_bits(f[3]) << 16);
+  v.z = float_to_bf16_bits(f[4]) | (float_to_bf16_bits(f[5]) << 16);
+  v.w = float_to_bf16_bits(f[6]) | (float_to_bf16_bits(f[7]) << 16);
+  *reinterpret_cast<uint4*>(p) = v;
+}
+__device__ __forceinline__ void st_vec(float* p, const float (&f)[8]) {
+  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  *reinterpret_cast<float4*>(p + 4) = make_float4(f[4], f[5], f[6], f[7]);
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -89,6 +122,14 @@ inline int check_dec_cache(const b200dec_cache* c, const b200kv_table* t) {
   if (t->max_pages < 1 || t->stride < 0) return B200KV_E_SHAPE;
   if (!aligned(c->k, 16) || !aligned(c->v, 16)) return B200KV_E_ALIGN;
   return B200KV_OK;
+}
+
+// sigmoid of an activation or output gate: in a bf16 model by the hardware's exponential and division (a few units of the
+// last 32-bit place), far below the bf16 rounding of what it multiplies
+template <typename T>
+__device__ __forceinline__ float sigmoid_act(float z) {
+  if constexpr (sizeof(T) == 4) return sigmoid_f(z);
+  else return __fdividef(1.f, 1.f + __expf(-fmaxf(z, -80.f)));  // the quotient is defined up to 2^126
 }
 
 // Device view of b200dec_attn_options (defaults filled in).

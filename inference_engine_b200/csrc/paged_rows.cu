@@ -122,14 +122,22 @@ rope_write_kernel(const T* __restrict__ qkv, long long qkv_stride, b200dec_rows 
 }
 
 // ---------------------------------------------------------------- norm of whole projections, interleaved rotation, write
-// One block per row.  kPairs: head sizes and the row stride are even, so channel pairs are loaded together.
+// One block per row; a thread owns channel pairs tid, tid + 256, ... of q | k | v.
 constexpr int kNrThreads = 256;
 
-template <typename T, bool kPairs>
+// Pair p of a group of heads of `pairs` pairs each (shift: log2 of it, or -1).
+__device__ __forceinline__ void nr_split(int p, int pairs, int shift, int& head, int& pr) {
+  head = shift >= 0 ? p >> shift : p / pairs;
+  pr = p - head * pairs;
+}
+
+// kKeep > 0: sizes and the row stride are even and a row has at most kKeep * 256 pairs, which stay in registers; their
+// weights and angles are loaded beside them.  0: any sizes, the row is read twice.
+template <typename T, int kKeep>
 __global__ void __launch_bounds__(kNrThreads)
 norm_rope_write_kernel(const T* __restrict__ qkv, long long qkv_stride, b200dec_rows rows, DecCache c, const float* __restrict__ q_norm,
                        const float* __restrict__ k_norm, float eps, const float* __restrict__ cos_sin, int table_len, int half, int heads,
-                       T* __restrict__ q_out, int32_t* status) {
+                       int k_shift, int v_shift, T* __restrict__ q_out, int32_t* status) {
   __shared__ float part[2][kNrThreads / 32];
   pdl_enter();
   const int r = blockIdx.x, tid = threadIdx.x;
@@ -152,85 +160,113 @@ norm_rope_write_kernel(const T* __restrict__ qkv, long long qkv_stride, b200dec_
     pos = 0;
   }
   const int page = ok ? dec_page(c, seq, pos, tid == 0 ? status : nullptr) : -1;
-  pdl_wait();
-  const T* src = qkv + r * qkv_stride;
-  const int nq = heads * c.k_dim, nk = c.heads * c.k_dim;
-  float sq = 0.f, sk = 0.f;
-  if (kPairs) {
-    for (int i = 2 * tid; i < nq + nk; i += 2 * kNrThreads) {
-      const float2 v = rw_load2(src + i);
-      const float s2 = fmaf(v.x, v.x, v.y * v.y);
-      if (i < nq) sq += s2; else sk += s2;
-    }
-  } else {
-    for (int i = tid; i < nq + nk; i += kNrThreads) {
-      const float v = ld_elem(src + i);
-      if (i < nq) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk);
-    }
-  }
-  sq = warp_sum(sq);
-  sk = warp_sum(sk);
-  if ((tid & 31) == 0) {
-    part[0][tid >> 5] = sq;
-    part[1][tid >> 5] = sk;
-  }
-  __syncthreads();
-  sq = sk = 0.f;
-#pragma unroll
-  for (int i = 0; i < kNrThreads / 32; ++i) {
-    sq += part[0][i];
-    sk += part[1][i];
-  }
-  const float inv_q = 1.0f / sqrtf(sq / (float)nq + eps), inv_k = 1.0f / sqrtf(sk / (float)nk + eps);
   const float2* cs = reinterpret_cast<const float2*>(cos_sin) + (long long)pos * half;
+  const T* src = qkv + r * qkv_stride;
+  const int nq = heads * c.k_dim, nk = c.heads * c.k_dim, all_heads = heads + c.heads;
+  const long long at0 = page < 0 ? 0 : dec_row(c, page, 0, pos % c.P);
   auto put2 = [](T* dst, float a, float b) {
     if (sizeof(T) == 2) *reinterpret_cast<uint32_t*>(dst) = float_to_bf16_bits(a) | (float_to_bf16_bits(b) << 16);
     else *reinterpret_cast<float2*>(dst) = make_float2(a, b);
   };
-  const int kpairs = c.k_row / 2, vpairs = c.v_row / 2;  // channels behind a size are written as zero
-  const long long at0 = page < 0 ? 0 : dec_row(c, page, 0, pos % c.P);
-  for (int i = tid; i < (heads + c.heads) * kpairs; i += kNrThreads) {
-    const int h = i / kpairs, pr = i - h * kpairs, ch = 2 * pr;
-    const bool is_q = h < heads;
-    if (!is_q && page < 0) continue;
-    float a = 0.f, b = 0.f;
-    if (ch < c.k_dim) {
-      const int off = h * c.k_dim + ch;  // q heads and k heads lie end to end
-      const float* w = is_q ? q_norm + off : k_norm + (off - nq);
-      const float inv = is_q ? inv_q : inv_k;
-      if (kPairs) {
-        const float2 v = rw_load2(src + off);
-        a = v.x * inv * w[0];
-        b = v.y * inv * w[1];
-      } else {
-        a = ld_elem(src + off) * inv * w[0];
-        if (ch + 1 < c.k_dim) b = ld_elem(src + off + 1) * inv * w[1];
+  // where channel ch of q / k head h (q heads first) goes; only for k heads a page is needed
+  auto place = [&](int h, int ch) {
+    return h < heads ? qdst + h * c.k_row + ch : (T*)c.k + (at0 + (long long)(h - heads) * c.P) * c.k_row + ch;
+  };
+  float sq = 0.f, sk = 0.f;
+  auto means = [&] {
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if ((tid & 31) == 0) {
+      part[0][tid >> 5] = sq;
+      part[1][tid >> 5] = sk;
+    }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < kNrThreads / 32; ++i) {
+      sq += part[0][i];
+      sk += part[1][i];
+    }
+    sq = 1.0f / sqrtf(sq / (float)nq + eps);
+    sk = 1.0f / sqrtf(sk / (float)nk + eps);
+  };
+  if constexpr (kKeep > 0) {
+    const int qkp = (nq + nk) / 2, all = qkp + c.heads * c.v_dim / 2;
+    float2 v[kKeep], w[kKeep], t[kKeep];
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {  // nothing here waits for the kernel in front
+      const int p = tid + i * kNrThreads;
+      if (p < qkp) {
+        int h, pr;
+        nr_split(p, c.k_dim / 2, k_shift, h, pr);
+        w[i] = *reinterpret_cast<const float2*>(2 * p < nq ? q_norm + 2 * p : k_norm + (2 * p - nq));
+        t[i] = pr < half ? cs[pr] : make_float2(1.f, 0.f);
       }
+    }
+    pdl_wait();
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+      const int p = tid + i * kNrThreads;
+      if (p < all) v[i] = rw_load2(src + 2 * p);
+    }
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+      const int p = tid + i * kNrThreads;
+      if (p < qkp) {
+        const float s2 = fmaf(v[i].x, v[i].x, v[i].y * v[i].y);
+        if (2 * p < nq) sq += s2; else sk += s2;
+      }
+    }
+    means();
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) {
+      const int p = tid + i * kNrThreads;
+      int h, pr;
+      if (p < qkp) {
+        nr_split(p, c.k_dim / 2, k_shift, h, pr);
+        if (h >= heads && page < 0) continue;
+        const float inv = h < heads ? sq : sk, a = v[i].x * inv * w[i].x, b = v[i].y * inv * w[i].y;
+        put2(place(h, 2 * pr), a * t[i].x - b * t[i].y, b * t[i].x + a * t[i].y);
+      } else if (p < all && page >= 0) {
+        nr_split(p - qkp, c.v_dim / 2, v_shift, h, pr);
+        put2((T*)c.v + (at0 + (long long)h * c.P) * c.v_row + 2 * pr, v[i].x, v[i].y);
+      }
+    }
+    // channels behind a size are written as zero
+    const int k_pad = (c.k_row - c.k_dim) / 2, v_pad = (c.v_row - c.v_dim) / 2;
+    for (int i = tid; i < all_heads * k_pad; i += kNrThreads)
+      if (i / k_pad < heads || page >= 0) put2(place(i / k_pad, c.k_dim + 2 * (i % k_pad)), 0.f, 0.f);
+    if (page >= 0)
+      for (int i = tid; i < c.heads * v_pad; i += kNrThreads)
+        put2((T*)c.v + (at0 + (long long)(i / v_pad) * c.P) * c.v_row + c.v_dim + 2 * (i % v_pad), 0.f, 0.f);
+  } else {
+    pdl_wait();
+    for (int i = tid; i < nq + nk; i += kNrThreads) {
+      const float f = ld_elem(src + i);
+      if (i < nq) sq = fmaf(f, f, sq); else sk = fmaf(f, f, sk);
+    }
+    means();
+    for (int i = tid; i < all_heads * (c.k_row / 2); i += kNrThreads) {
+      const int h = i / (c.k_row / 2), pr = i - h * (c.k_row / 2), ch = 2 * pr, off = h * c.k_dim + ch;  // q and k heads lie end to end
+      if (h >= heads && page < 0) continue;
+      const float* w = h < heads ? q_norm + off : k_norm + (off - nq);
+      const float inv = h < heads ? sq : sk;
+      float a = ch < c.k_dim ? ld_elem(src + off) * inv * w[0] : 0.f;
+      float b = ch + 1 < c.k_dim ? ld_elem(src + off + 1) * inv * w[1] : 0.f;
       if (pr < half) {
         const float2 t = cs[pr];
-        const float u = a, v = b;
-        a = u * t.x - v * t.y;
-        b = v * t.x + u * t.y;
+        const float u = a;
+        a = u * t.x - b * t.y;
+        b = b * t.x + u * t.y;
       }
+      put2(place(h, ch), a, b);
     }
-    put2(is_q ? qdst + h * c.k_row + ch : (T*)c.k + (at0 + (long long)(h - heads) * c.P) * c.k_row + ch, a, b);
-  }
-  if (page < 0) return;
-  const T* vsrc = src + nq + nk;
-  for (int i = tid; i < c.heads * vpairs; i += kNrThreads) {
-    const int h = i / vpairs, ch = 2 * (i - h * vpairs);
-    float a = 0.f, b = 0.f;
-    if (ch < c.v_dim) {
-      if (kPairs) {
-        const float2 v = rw_load2(vsrc + h * c.v_dim + ch);
-        a = v.x;
-        b = v.y;
-      } else {
-        a = ld_elem(vsrc + h * c.v_dim + ch);
-        if (ch + 1 < c.v_dim) b = ld_elem(vsrc + h * c.v_dim + ch + 1);
-      }
+    if (page < 0) return;
+    for (int i = tid; i < c.heads * (c.v_row / 2); i += kNrThreads) {
+      const int h = i / (c.v_row / 2), ch = 2 * (i - h * (c.v_row / 2));
+      const T* p = src + nq + nk + h * c.v_dim + ch;
+      put2((T*)c.v + (at0 + (long long)h * c.P) * c.v_row + ch, ch < c.v_dim ? ld_elem(p) : 0.f, ch + 1 < c.v_dim ? ld_elem(p + 1) : 0.f);
     }
-    put2((T*)c.v + (at0 + (long long)h * c.P) * c.v_row + ch, a, b);
   }
 }
 
@@ -383,14 +419,29 @@ extern "C" int b200dec_norm_rope_write(const void* qkv, int64_t qkv_stride, cons
   if (!aligned(q_out, 16) || !aligned(cos_sin, 8)) return B200KV_E_ALIGN;
   const DecCache c = dec_view(cache, table);
   cudaStream_t s = (cudaStream_t)stream;
-  const bool pairs = cache->k_dim % 2 == 0 && cache->v_dim % 2 == 0 && qkv_stride % 2 == 0 && aligned(qkv, 2 * cache->elem);
+  const bool even = cache->k_dim % 2 == 0 && cache->v_dim % 2 == 0 && qkv_stride % 2 == 0 && aligned(qkv, 2 * cache->elem) &&
+                    aligned(q_norm, 8) && aligned(k_norm, 8);
+  const long long pairs = ((long long)(heads + cache->kv_heads) * cache->k_dim + (long long)cache->kv_heads * cache->v_dim) / 2;
+  auto log2_of = [](int n) {
+    for (int i = 0; i < 30; ++i)
+      if (n == 1 << i) return i;
+    return -1;
+  };
   auto run = [&](auto* kernel, auto* in, auto* q) {
     return launch_result(launch_chained(kernel, dim3(rows->num_rows), dim3(kNrThreads), 0, s, in, (long long)qkv_stride, *rows, c, q_norm,
-                                        k_norm, eps, cos_sin, table_len, half, heads, q, status));
+                                        k_norm, eps, cos_sin, table_len, half, heads, log2_of(cache->k_dim / 2), log2_of(cache->v_dim / 2), q,
+                                        status));
   };
+  const int keep = !even ? 0 : pairs <= 4 * kNrThreads ? 4 : pairs <= 8 * kNrThreads ? 8 : pairs <= 16 * kNrThreads ? 16 : 0;
   if (cache->elem == 2)
-    return run(pairs ? norm_rope_write_kernel<uint16_t, true> : norm_rope_write_kernel<uint16_t, false>, (const uint16_t*)qkv, (uint16_t*)q_out);
-  return run(pairs ? norm_rope_write_kernel<float, true> : norm_rope_write_kernel<float, false>, (const float*)qkv, (float*)q_out);
+    return run(keep == 4   ? norm_rope_write_kernel<uint16_t, 4>
+               : keep == 8 ? norm_rope_write_kernel<uint16_t, 8>
+               : keep      ? norm_rope_write_kernel<uint16_t, 16> : norm_rope_write_kernel<uint16_t, 0>,
+               (const uint16_t*)qkv, (uint16_t*)q_out);
+  return run(keep == 4   ? norm_rope_write_kernel<float, 4>
+             : keep == 8 ? norm_rope_write_kernel<float, 8>
+             : keep      ? norm_rope_write_kernel<float, 16> : norm_rope_write_kernel<float, 0>,
+             (const float*)qkv, (float*)q_out);
 }
 
 extern "C" int b200dec_attn_rows_opt(const void* q, const b200dec_cache* cache, const b200kv_table* table, const b200dec_rows* rows,

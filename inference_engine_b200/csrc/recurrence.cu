@@ -36,7 +36,7 @@ __device__ __forceinline__ float rd_sum(float v, float* part) {
 // Threads are laid out as `rg` groups of rows by `cg` columns of four state entries; a thread owns rows r, r + rg, ...
 // kRows > 0: its entries stay in registers between the reduction and the update; 0: any size, the state is read twice.
 template <typename T, int kRows>
-__global__ void __launch_bounds__(kRdThreads)
+__global__ void __launch_bounds__(kRdThreads, kRows <= 4 ? 4 : (kRows <= 8 ? 3 : 2))
 recurrence_decode_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, const b200dec_entries ent, const RecNorm norm,
                          void* __restrict__ out, int cg, int rg, int32_t* status) {
   extern __shared__ __align__(16) float rd_smem[];
@@ -50,7 +50,7 @@ recurrence_decode_kernel(const b200dec_recurrence rec, const b200dec_recurrence_
   float* us = vs + P4;                 // [P4]
   float* os = us + P4;                 // [P4]
   float* red = os + P4;                // [2][rg][4 * cg]
-  __shared__ float part[kRdThreads / 32];
+  __shared__ float part[3 * kRdThreads / 32];
   const int nd = min(*ent.num_decoding, ent.num_entries);
   if (e >= nd) {  // idle; in a pure decode step the row is cleared
     pdl_wait();
@@ -76,61 +76,105 @@ recurrence_decode_kernel(const b200dec_recurrence rec, const b200dec_recurrence_
       if (mine && d < D && x.pos > 0) S[i] = __ldcg(reinterpret_cast<const float4*>(state + (long long)d * P4) + c4);
     }
   }
-  // ---- the token's q, k, v (convolution and silu), decays and step
+  // ---- the token's q, k, v (convolution and silu), decays and step; two channels per thread at a time, all loads of
+  // both ahead of the arithmetic
   const int per = rec.heads / rec.qk_heads, hq = h / per;
   const T* xr = (const T*)in.x + x.first * in.x_stride;
+  const T* sr = (const T*)in.step + x.first * in.step_stride;
   T* ring = (T*)rec.ring + (long long)x.slot * rec.taps * rec.channels;
-  const int now = x.pos % rec.taps;
+  const int now = x.pos % rec.taps, back = min(rec.taps - 1, x.pos);
   const bool first_of_group = h % per == 0;
-  auto conv = [&](int ch, bool keep) {
-    const T raw = xr[ch];
-    if (keep) ring[(long long)now * rec.channels + ch] = raw;
-    return rec_conv(rec, ch, x.pos, ld_elem(&raw), [&](int j) {
-      int at = now - j;
-      if (at < 0) at += rec.taps;
-      return ldcg_elem(ring + (long long)at * rec.channels + ch);
-    });
-  };
   const float na = rec.neg_a[h];
   float step = 0.f;
-  if (!rec.channel_decay) step = softplus_f(ld_elem((const T*)in.step + x.first * in.step_stride + h) + rec.dt_bias[h]);
-  const float decay_all = expf(na * step);
+  if (!rec.channel_decay) step = ld_elem(sr + h) + rec.dt_bias[h];
+  const float beta_in = rec.correct ? ld_elem((const T*)in.beta + x.first * in.beta_stride + h) : 0.f;
   float sq = 0.f, sk = 0.f, qk = 0.f;
-  for (int i = tid; i < 2 * Dp + P4; i += kRdThreads) {
-    if (i < 2 * Dp) {
-      const bool is_q = i < Dp;
-      const int d = is_q ? i : i - Dp;
-      float v = 0.f;
-      if (d < D) v = conv((is_q ? rec.off_q : rec.off_k) + hq * D + d, first_of_group);
-      (is_q ? qs : ks)[d] = v;
-      if (is_q) sq = fmaf(v, v, sq);
-      else {
-        sk = fmaf(v, v, sk);
-        float g = decay_all;
-        if (rec.channel_decay && d < D)
-          g = expf(na * softplus_f(ld_elem((const T*)in.step + x.first * in.step_stride + h * D + d) + rec.dt_bias[h * D + d]));
-        gs[d] = g;
+  const int total = 2 * Dp + P4;
+  constexpr int kNear = 4;  // taps handled without a loop
+  for (int base = tid; base < total; base += 2 * kRdThreads) {
+    float xv[2][kNear], wv[2][kNear], bv[2], dv[2];
+    int ch[2];
+    T raw[2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = base + u * kRdThreads, d = i < Dp ? i : i - Dp;
+      ch[u] = -1;
+      if (i < Dp) { if (d < D) ch[u] = rec.off_q + hq * D + d; }
+      else if (i < 2 * Dp) { if (d < D) ch[u] = rec.off_k + hq * D + d; }
+      else if (i < total && i - 2 * Dp < P) ch[u] = rec.off_v + h * P + i - 2 * Dp;
+      if (ch[u] < 0) continue;
+      raw[u] = xr[ch[u]];
+      bv[u] = rec.conv_b ? rec.conv_b[ch[u]] : 0.f;
+      dv[u] = 0.f;
+      if (rec.channel_decay && i >= Dp && i < 2 * Dp) dv[u] = ld_elem(sr + h * D + d) + rec.dt_bias[h * D + d];
+#pragma unroll
+      for (int j = 0; j < kNear; ++j) {
+        xv[u][j] = wv[u][j] = 0.f;
+        if (j > back) continue;
+        int at = now - j;
+        if (at < 0) at += rec.taps;
+        wv[u][j] = rec.conv_w[(long long)(rec.taps - 1 - j) * rec.channels + ch[u]];
+        if (j > 0) xv[u][j] = ldcg_elem(ring + (long long)at * rec.channels + ch[u]);
       }
-    } else {
-      const int p = i - 2 * Dp;
-      vs[p] = p < P ? conv(rec.off_v + h * P + p, true) : 0.f;
+    }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int i = base + u * kRdThreads;
+      if (i >= total) break;
+      float v = 0.f;
+      if (ch[u] >= 0) {
+        xv[u][0] = ld_elem(&raw[u]);
+        v = bv[u];
+#pragma unroll
+        for (int j = 0; j < kNear; ++j) v = fmaf(wv[u][j], xv[u][j], v);
+        for (int j = kNear; j <= back; ++j) {
+          int at = now - j;
+          if (at < 0) at += rec.taps;
+          v = fmaf(rec.conv_w[(long long)(rec.taps - 1 - j) * rec.channels + ch[u]], ldcg_elem(ring + (long long)at * rec.channels + ch[u]), v);
+        }
+        v *= sigmoid_act<T>(v);
+        if (i >= 2 * Dp || first_of_group) ring[(long long)now * rec.channels + ch[u]] = raw[u];
+      }
+      if (i < Dp) {
+        qs[i] = v;
+        sq = fmaf(v, v, sq);
+      } else if (i < 2 * Dp) {
+        ks[i - Dp] = v;
+        sk = fmaf(v, v, sk);
+        if (rec.channel_decay) gs[i - Dp] = ch[u] >= 0 ? expf(na * softplus_f(dv[u])) : 1.f;
+      } else {
+        vs[i - 2 * Dp] = v;
+      }
     }
   }
-  if (rec.unit_norm) {
-    sq = rd_sum(sq, part);
-    sk = rd_sum(sk, part);
-  } else {
-    __syncthreads();
+  if (!rec.channel_decay) {
+    step = softplus_f(step);
+    const float g = expf(na * step);
+    for (int d = tid; d < Dp; d += kRdThreads) gs[d] = g;
   }
+  __syncthreads();
+  for (int d = tid; d < D; d += kRdThreads) qk = fmaf(qs[d], ks[d], qk);
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  qk = warp_sum(qk);
+  if ((tid & 31) == 0) {
+    part[tid >> 5] = sq;
+    part[8 + (tid >> 5)] = sk;
+    part[16 + (tid >> 5)] = qk;
+  }
+  __syncthreads();
+  sq = sk = qk = 0.f;
+#pragma unroll
+  for (int i = 0; i < kRdThreads / 32; ++i) {
+    sq += part[i];
+    sk += part[8 + i];
+    qk += part[16 + i];
+  }
+  // the factors of q and k are applied to the sums, not to the vectors
   const float fq = rec.q_scale * (rec.unit_norm ? 1.0f / sqrtf(sq + rec.unit_eps) : 1.f);
   const float fk = rec.unit_norm ? 1.0f / sqrtf(sk + rec.unit_eps) : 1.f;
-  for (int d = tid; d < D; d += kRdThreads) {
-    qs[d] *= fq;
-    ks[d] *= fk;
-    qk = fmaf(qs[d], ks[d], qk);
-  }
-  qk = rd_sum(qk, part);
-  const float beta = rec.correct ? sigmoid_f(ld_elem((const T*)in.beta + x.first * in.beta_stride + h)) : step;
+  qk *= fq * fk;
+  const float beta = rec.correct ? sigmoid_f(beta_in) : step;
   const float skip = rec.skip ? rec.skip[h] : 0.f;
   // ---- (decay S)^T k and (decay S)^T q, then the update, in slabs of 4 * cg columns
   float ss = 0.f;
@@ -161,14 +205,15 @@ recurrence_decode_kernel(const b200dec_recurrence rec, const b200dec_recurrence_
     __syncthreads();
     for (int i = tid; i < 4 * cg && col0 + i < P4; i += kRdThreads) {
       float rk = 0.f, rq = 0.f;
+#pragma unroll 8
       for (int r = 0; r < rg; ++r) {
         rk += red[r * 4 * cg + i];
         rq += red[(rg + r) * 4 * cg + i];
       }
       const float v = vs[col0 + i];
-      const float u = rec.correct ? beta * (v - rk) : beta * v;
-      us[col0 + i] = u;
-      const float o = fmaf(skip, v, fmaf(qk, u, rq));
+      const float u = rec.correct ? beta * fmaf(-fk, rk, v) : beta * v;
+      us[col0 + i] = fk * u;
+      const float o = fmaf(skip, v, fmaf(qk, u, fq * rq));
       os[col0 + i] = o;
       ss = fmaf(o, o, ss);
     }
@@ -207,78 +252,101 @@ recurrence_decode_kernel(const b200dec_recurrence rec, const b200dec_recurrence_
 }
 
 // ---------------------------------------------------------------- convolution of prompt portions
-constexpr int kRcThreads = 256;
+constexpr int kRcThreads = 128;
+constexpr int kRcRun = 8;  // rows per thread
 
-// kVec channels (8, or 1 for any size) of one row per thread.
-template <typename T, int kVec>
+// kVec channels (8, or 1 for any size) of kRcRun consecutive rows per thread.  kTaps > 0: the taps' weights and the rows'
+// inputs are held in registers, so that every input is loaded once.  kTaps = 0: any number of taps, row by row.
+template <typename T, int kVec, int kTaps>
 __global__ void __launch_bounds__(kRcThreads)
 conv_rows_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, const b200dec_entries ent, T* __restrict__ out,
                  int out_stride, int32_t* status) {
   pdl_enter();
-  const int r = blockIdx.y, ch = (blockIdx.x * kRcThreads + threadIdx.x) * kVec;
-  const int e = ent.seq_ids[r];
-  if (e < *ent.num_decoding || e >= ent.num_entries || ch >= rec.channels) return;
-  const int pos = ent.positions[r], first = ent.cu_seqlens[e], slot = ent.slots[e];
-  if (slot < 0 || slot >= rec.num_slots || pos < 0 || first < 0 || first > r) {
-    if (slot != -1 && threadIdx.x == 0 && status) atomicOr(status, B200KV_S_BAD_POSITION);
-    return;
-  }
+  const int r0 = blockIdx.x * kRcRun, ch = (blockIdx.y * kRcThreads + threadIdx.x) * kVec;
+  if (ch >= rec.channels) return;
+  const int nd = *ent.num_decoding;
+  constexpr int kHold = kTaps > 0 ? kTaps : 1;
+  float w[kHold][kVec], bias[kVec];
+#pragma unroll
+  for (int i = 0; i < kVec; ++i) bias[i] = rec.conv_b ? rec.conv_b[ch + i] : 0.f;
+  if (kTaps > 0)
+#pragma unroll
+    for (int j = 0; j < kHold; ++j) ld_vec(rec.conv_w + (long long)j * rec.channels + ch, w[j]);
   pdl_wait();
-  const T* ring = (const T*)rec.ring + (long long)slot * rec.taps * rec.channels + ch;
-  float acc[kVec], f[kVec];
-  auto load = [&](const T* p, bool fresh) {
-    if constexpr (kVec == 1) {
-      f[0] = fresh ? ldcg_elem(p) : ld_elem(p);
+  // Input j positions before row r (of an entry whose rows start at `first`), zero in front of the sequence.
+  auto before = [&](int r, int j, int first, int pos, int slot, float (&f)[kVec]) {
+    if (j > pos) {
+#pragma unroll
+      for (int i = 0; i < kVec; ++i) f[i] = 0.f;
+    } else if (r - j >= first) {
+      ld_vec((const T*)in.x + (long long)(r - j) * in.x_stride + ch, f);
     } else {
+      const T* p = (const T*)rec.ring + ((long long)slot * rec.taps + (pos - j) % rec.taps) * rec.channels + ch;
+      if constexpr (kVec == 1) {
+        f[0] = ldcg_elem(p);
+      } else if constexpr (sizeof(T) == 2) {
+        unpack8(__ldcg(reinterpret_cast<const uint4*>(p)), f);
+      } else {
+        float a[4], b[4];
+        ld_fresh4(p, a);
+        ld_fresh4(p + 4, b);
 #pragma unroll
-      for (int i = 0; i < kVec; i += 4) {
-        float t[4];
-        if constexpr (sizeof(T) == 2) {
-          const uint2 v = fresh ? __ldcg(reinterpret_cast<const uint2*>(p + i)) : *reinterpret_cast<const uint2*>(p + i);
-          t[0] = __uint_as_float(v.x << 16); t[1] = __uint_as_float(v.x & 0xFFFF0000u);
-          t[2] = __uint_as_float(v.y << 16); t[3] = __uint_as_float(v.y & 0xFFFF0000u);
-        } else {
-          ld_fresh4(p + i, t);
-        }
-#pragma unroll
-        for (int k = 0; k < 4; ++k) f[i + k] = t[k];
+        for (int i = 0; i < 4; ++i) { f[i] = a[i]; f[4 + i] = b[i]; }
       }
     }
   };
+  auto put = [&](int r, float (&acc)[kVec]) {
 #pragma unroll
-  for (int i = 0; i < kVec; ++i) acc[i] = rec.conv_b ? rec.conv_b[ch + i] : 0.f;
-  const int back = min(rec.taps - 1, pos);
-  for (int j = 0; j <= back; ++j) {
-    if (r - j >= first) load((const T*)in.x + (long long)(r - j) * in.x_stride + ch, false);
-    else load(ring + (long long)((pos - j) % rec.taps) * rec.channels, true);
-    const float* w = rec.conv_w + (long long)(rec.taps - 1 - j) * rec.channels + ch;
+    for (int i = 0; i < kVec; ++i) acc[i] *= sigmoid_act<T>(acc[i]);
+    st_vec(out + (long long)r * out_stride + ch, acc);
+  };
+  const int rows = min(kRcRun, ent.num_rows - r0);
+  float x[kRcRun + kHold - 1][kVec];  // inputs of rows r0 - (taps - 1) .. r0 + kRcRun - 1, as the entry at hand sees them
+  if (kTaps > 0) {
 #pragma unroll
-    for (int i = 0; i < kVec; ++i) acc[i] = fmaf(w[i], f[i], acc[i]);
+    for (int t = 0; t < kRcRun; ++t)
+      if (t < rows) ld_vec((const T*)in.x + (long long)(r0 + t) * in.x_stride + ch, x[t + kHold - 1]);
   }
-  T* dst = out + (long long)r * out_stride + ch;
+  int e_last = -1;
 #pragma unroll
-  for (int i = 0; i < kVec; ++i) acc[i] = silu_f(acc[i]);
-  if constexpr (kVec == 1) {
-    st_elem(dst, acc[0]);
-  } else {
-#pragma unroll
-    for (int i = 0; i < kVec; i += 4) {
-      const float t[4] = {acc[i], acc[i + 1], acc[i + 2], acc[i + 3]};
-      st_elem4(dst + i, t);
+  for (int t = 0; t < kRcRun; ++t) {
+    if (t >= rows) break;
+    const int r = r0 + t, e = ent.seq_ids[r];
+    const bool fresh = e != e_last;
+    e_last = e;
+    if (e < nd || e >= ent.num_entries) continue;
+    const int pos = ent.positions[r], first = ent.cu_seqlens[e], slot = ent.slots[e];
+    if (slot < 0 || slot >= rec.num_slots || pos < 0 || first < 0 || first > r) {
+      if (slot != -1 && ch == 0 && status) atomicOr(status, B200KV_S_BAD_POSITION);
+      continue;
     }
-  }
-}
-
-// The raw inputs of the last `taps` positions of an entry's portion go into its ring; block `part` of `parts` does its share.
-template <typename T>
-__device__ __forceinline__ void rec_keep_inputs(const b200dec_recurrence& rec, const b200dec_recurrence_in& in, const RecEntry& x, int part,
-                                                int parts, int threads) {
-  const int keep = min(rec.taps, x.n);
-  T* ring = (T*)rec.ring + (long long)x.slot * rec.taps * rec.channels;
-  for (int j = 0; j < keep; ++j) {
-    const int row = x.first + x.n - 1 - j, at = (x.pos + x.n - 1 - j) % rec.taps;
-    for (int c = part * threads + threadIdx.x; c < rec.channels; c += parts * threads)
-      ring[(long long)at * rec.channels + c] = ((const T*)in.x)[row * in.x_stride + c];
+    float acc[kVec];
+#pragma unroll
+    for (int i = 0; i < kVec; ++i) acc[i] = bias[i];
+    if (kTaps > 0) {
+      float h[kHold][kVec];
+      if (fresh) {  // the first row of the thread or of an entry: its history comes from elsewhere
+#pragma unroll
+        for (int j = 1; j < kHold; ++j) before(r, j, first, pos, slot, h[j]);
+      }
+#pragma unroll
+      for (int j = 1; j < kHold; ++j)
+#pragma unroll
+        for (int i = 0; i < kVec; ++i) {
+          if (fresh) x[t + kHold - 1 - j][i] = h[j][i];
+          acc[i] = fmaf(w[kHold - 1 - j][i], x[t + kHold - 1 - j][i], acc[i]);
+        }
+#pragma unroll
+      for (int i = 0; i < kVec; ++i) acc[i] = fmaf(w[kHold - 1][i], x[t + kHold - 1][i], acc[i]);
+    } else {
+      for (int j = 0; j < rec.taps; ++j) {
+        float f[kVec];
+        before(r, j, first, pos, slot, f);
+#pragma unroll
+        for (int i = 0; i < kVec; ++i) acc[i] = fmaf(rec.conv_w[(long long)(rec.taps - 1 - j) * rec.channels + ch + i], f[i], acc[i]);
+      }
+    }
+    put(r, acc);
   }
 }
 
@@ -450,10 +518,12 @@ template <typename T>
 static int rc_run(const b200dec_recurrence& rec, const b200dec_recurrence_in& in, const b200dec_entries& ent, void* out, int32_t* status,
                   cudaStream_t s) {
   const bool vec = rec.channels % 8 == 0 && in.x_stride % 8 == 0 && aligned(in.x, 16) && aligned(rec.ring, 16) && aligned(out, 16);
-  const int items = vec ? rec.channels / 8 : rec.channels;
-  auto* kernel = vec ? conv_rows_kernel<T, 8> : conv_rows_kernel<T, 1>;
-  return launch_result(launch_chained(kernel, dim3((items + kRcThreads - 1) / kRcThreads, ent.num_rows), dim3(kRcThreads), 0, s, rec, in, ent,
-                                      (T*)out, (rec.channels + 7) / 8 * 8, status));
+  const dim3 grid((ent.num_rows + kRcRun - 1) / kRcRun, ((vec ? rec.channels / 8 : rec.channels) + kRcThreads - 1) / kRcThreads);
+  auto* kernel = vec ? (rec.taps == 4   ? conv_rows_kernel<T, 8, 4>
+                        : rec.taps == 3 ? conv_rows_kernel<T, 8, 3>
+                        : rec.taps == 2 ? conv_rows_kernel<T, 8, 2> : conv_rows_kernel<T, 8, 0>)
+                     : conv_rows_kernel<T, 1, 0>;
+  return launch_result(launch_chained(kernel, grid, dim3(kRcThreads), 0, s, rec, in, ent, (T*)out, (rec.channels + 7) / 8 * 8, status));
 }
 
 }  // namespace b200kv
@@ -478,7 +548,6 @@ extern "C" int b200dec_conv_rows(const b200dec_recurrence* rec, const b200dec_re
   if (rc != B200KV_OK) return rc;
   if (!ent->cu_seqlens || !conv_out) return B200KV_E_NULL;
   if (ent->num_rows == 0) return B200KV_OK;
-  if (ent->num_rows > 65535) return B200KV_E_RANGE;
   cudaStream_t s = (cudaStream_t)stream;
   return rec->elem == 2 ? rc_run<uint16_t>(*rec, *in, *ent, conv_out, status, s) : rc_run<float>(*rec, *in, *ent, conv_out, status, s);
 }

@@ -28,19 +28,21 @@ __device__ __forceinline__ RecEntry rec_entry(const b200dec_entries& ent, const 
 
 __host__ __device__ constexpr int rec_round4(int n) { return (n + 3) / 4 * 4; }
 
-// silu of the causal convolution of channel ch at position pos; `cur` = the token's own input, before(j) = the input j
-// positions earlier (only asked for positions >= 0).
-template <typename Before>
-__device__ __forceinline__ float rec_conv(const b200dec_recurrence& rec, int ch, int pos, float cur, Before before) {
-  float acc = rec.conv_b ? rec.conv_b[ch] : 0.f;
-  acc = fmaf(rec.conv_w[(long long)(rec.taps - 1) * rec.channels + ch], cur, acc);
-  const int back = min(rec.taps - 1, pos);
-  for (int j = 1; j <= back; ++j) acc = fmaf(rec.conv_w[(long long)(rec.taps - 1 - j) * rec.channels + ch], before(j), acc);
-  return silu_f(acc);
-}
-
 __device__ __forceinline__ float ldcg_elem(const uint16_t* p) { return bf16_bits_to_float(__ldcg(p)); }
 __device__ __forceinline__ float ldcg_elem(const float* p) { return __ldcg(p); }
+
+// The raw inputs of the last `taps` positions of an entry's portion go into its ring; block `part` of `parts` does its share.
+template <typename T>
+__device__ __forceinline__ void rec_keep_inputs(const b200dec_recurrence& rec, const b200dec_recurrence_in& in, const RecEntry& x, int part,
+                                                int parts, int threads) {
+  const int keep = min(rec.taps, x.n);
+  T* ring = (T*)rec.ring + (long long)x.slot * rec.taps * rec.channels;
+  for (int j = 0; j < keep; ++j) {
+    const int row = x.first + x.n - 1 - j, at = (x.pos + x.n - 1 - j) % rec.taps;
+    for (int c = part * threads + threadIdx.x; c < rec.channels; c += parts * threads)
+      ring[(long long)at * rec.channels + c] = ((const T*)in.x)[row * in.x_stride + c];
+  }
+}
 
 inline int check_recurrence(const b200dec_recurrence* r, const b200dec_recurrence_in* in, const b200dec_entries* e) {
   if (!r || !in || !e || !r->state || !r->ring || !r->conv_w || !r->neg_a || !r->dt_bias || !in->x || !in->step) return B200KV_E_NULL;

@@ -173,31 +173,27 @@ norm_add_kernel(float* x, const T* __restrict__ y, const float* __restrict__ wei
   }
 }
 
-template <typename T>
+// kVec channels (8, or 1 for any size) of one row per thread.
+template <typename T, int kVec>
 __global__ void __launch_bounds__(kRowThreads)
-silu_mul_rows_kernel(const T* __restrict__ gu, long long stride, T* __restrict__ out, long long out_stride, int rows, int ff, int vec) {
+silu_mul_rows_kernel(const T* __restrict__ gu, long long stride, T* __restrict__ out, long long out_stride, int rows, int ff) {
   pdl_enter();
   pdl_wait();
-  const int per = vec ? ff / 4 : ff;
-  const long long i = (long long)blockIdx.x * kRowThreads + threadIdx.x;
-  if (i >= (long long)rows * per) return;
-  const int r = (int)(i / per), c = (int)(i - (long long)r * per);
-  const T* src = gu + r * stride;
-  if (vec) {
-    float g[4], u[4];
-    ld_elem4(src + 4 * c, g);
-    ld_elem4(src + ff + 4 * c, u);
+  const long long r = blockIdx.x;
+  const int c = (blockIdx.y * kRowThreads + threadIdx.x) * kVec;
+  if (c >= ff) return;
+  const T* src = gu + r * stride + c;
+  float g[kVec], u[kVec];
+  ld_vec(src, g);
+  ld_vec(src + ff, u);
 #pragma unroll
-    for (int e = 0; e < 4; ++e) g[e] = silu_f(g[e]) * u[e];
-    st_elem4(out + r * out_stride + 4 * c, g);
-  } else {
-    st_elem(out + r * out_stride + c, silu_f(ld_elem(src + c)) * ld_elem(src + ff + c));
-  }
+  for (int e = 0; e < kVec; ++e) g[e] = g[e] * sigmoid_act<T>(g[e]) * u[e];
+  st_vec(out + r * out_stride + c, g);
 }
 
-// Norm of every part of a row by itself, with a gate before or after: kThreads threads per part (a warp or the block),
-// kKeep channels of it in registers per thread (0: read twice).
-template <typename T, int kThreads, int kKeep>
+// Norm of every part of a row by itself with a gate before or after: kThreads threads per part (a warp or the block), kVec
+// neighbouring channels at a time, kKeep such groups in registers per thread (0: read twice).
+template <typename T, int kThreads, int kVec, int kKeep>
 __global__ void __launch_bounds__(kRowThreads)
 gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long long gate_stride, int gate_first,
                   const float* __restrict__ weight, int weight_len, float eps, float out_scale, T* __restrict__ out, long long out_stride,
@@ -212,37 +208,58 @@ gated_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, long 
   const float* src = o + (long long)r * len + p * part;
   const T* g = gate + r * gate_stride + p * part;
   T* dst = out + r * out_stride + p * part;
-  auto value = [&](int c) { return gate_first ? src[c] * silu_f(ld_elem(g + c)) : src[c]; };
-  float keep[kKeep > 0 ? kKeep : 1], ss = 0.f;
+  // v: the value before the norm, f: what it is multiplied by behind it
+  auto load = [&](int c, float (&v)[kVec], float (&f)[kVec]) {
+    float z[kVec];
+    ld_vec(src + c, v);
+    ld_vec(g + c, z);
+#pragma unroll
+    for (int i = 0; i < kVec; ++i) {
+      const float s = sigmoid_act<T>(z[i]);
+      f[i] = gate_first ? 1.f : s;
+      if (gate_first) v[i] *= z[i] * s;
+    }
+  };
+  auto put = [&](int c, float inv, float (&v)[kVec], const float (&f)[kVec]) {
+#pragma unroll
+    for (int i = 0; i < kVec; ++i) {
+      const int at = p * part + c + i;
+      v[i] = v[i] * inv * weight[weight_len == len ? at : at % weight_len] * f[i] * out_scale;
+    }
+    st_vec(dst + c, v);
+  };
+  float v[kKeep > 0 ? kKeep : 1][kVec], f[kKeep > 0 ? kKeep : 1][kVec], ss = 0.f;
   if (live) {
     if (kKeep > 0) {
 #pragma unroll
       for (int i = 0; i < kKeep; ++i) {
-        const int c = t + i * kThreads;
-        keep[i] = c < part ? value(c) : 0.f;
-        ss = fmaf(keep[i], keep[i], ss);
+        const int c = (t + i * kThreads) * kVec;
+        if (c < part) {
+          load(c, v[i], f[i]);
+#pragma unroll
+          for (int k = 0; k < kVec; ++k) ss = fmaf(v[i][k], v[i][k], ss);
+        }
       }
     } else {
-      for (int c = t; c < part; c += kThreads) {
-        const float v = value(c);
-        ss = fmaf(v, v, ss);
+      for (int c = t * kVec; c < part; c += kThreads * kVec) {
+        load(c, v[0], f[0]);
+#pragma unroll
+        for (int k = 0; k < kVec; ++k) ss = fmaf(v[0][k], v[0][k], ss);
       }
     }
   }
   ss = kThreads == 32 ? warp_sum(ss) : row_sum(ss);
   if (!live) return;
   const float inv = 1.0f / sqrtf(ss / (float)part + eps);
-  auto put = [&](int c, float v) {
-    const int at = p * part + c;
-    v = v * inv * weight[weight_len == len ? at : at % weight_len] * out_scale;
-    st_elem(dst + c, gate_first ? v : v * sigmoid_f(ld_elem(g + c)));
-  };
   if (kKeep > 0) {
 #pragma unroll
     for (int i = 0; i < kKeep; ++i)
-      if (t + i * kThreads < part) put(t + i * kThreads, keep[i]);
+      if ((t + i * kThreads) * kVec < part) put((t + i * kThreads) * kVec, inv, v[i], f[i]);
   } else {
-    for (int c = t; c < part; c += kThreads) put(c, value(c));
+    for (int c = t * kVec; c < part; c += kThreads * kVec) {
+      load(c, v[0], f[0]);
+      put(c, inv, v[0], f[0]);
+    }
   }
 }
 
@@ -259,10 +276,15 @@ static int run_gated_norm(const float* o, const void* gate, int64_t gate_stride,
                           float eps, float out_scale, void* out, int64_t out_stride, int rows, int len, int parts,
                           cudaStream_t s) {
   const int part = len / parts;
-  const bool warp = part <= 32 * 8;
-  auto* kernel = part <= 128 ? gated_norm_kernel<T, 32, 4> : warp ? gated_norm_kernel<T, 32, 8>
-                 : part <= kRowThreads * 8 ? gated_norm_kernel<T, kRowThreads, 8>
-                 : part <= kRowThreads * 16 ? gated_norm_kernel<T, kRowThreads, 16> : gated_norm_kernel<T, kRowThreads, 0>;
+  const bool vec = part % 4 == 0 && len % 4 == 0 && gate_stride % 4 == 0 && out_stride % 4 == 0 && aligned(o, 16) && aligned(gate, 16) &&
+                   aligned(out, 16);
+  const bool warp = part <= (vec ? 512 : 256);
+  auto* kernel = vec ? (part <= 128   ? gated_norm_kernel<T, 32, 4, 1>
+                        : warp        ? gated_norm_kernel<T, 32, 4, 4>
+                        : part <= 1024 ? gated_norm_kernel<T, kRowThreads, 4, 1>
+                        : part <= 4096 ? gated_norm_kernel<T, kRowThreads, 4, 4>
+                                       : gated_norm_kernel<T, kRowThreads, 4, 0>)
+                     : (warp ? gated_norm_kernel<T, 32, 1, 8> : gated_norm_kernel<T, kRowThreads, 1, 0>);
   const long long items = (long long)rows * parts, per = warp ? kRowThreads / 32 : 1, blocks = (items + per - 1) / per;
   if (blocks > 0x7FFFFFF0ll) return B200KV_E_RANGE;
   return launch_result(launch_chained(kernel, dim3((unsigned)blocks), dim3(kRowThreads), 0, s, o, (const T*)gate, (long long)gate_stride,
@@ -335,15 +357,14 @@ extern "C" int b200dec_silu_mul(const void* gate_up, int64_t stride, int32_t ele
   if (num_rows == 0) return B200KV_OK;
   if (!gate_up || !out) return B200KV_E_NULL;
   if (num_rows < 0 || ff < 1 || stride < 2 * (int64_t)ff || out_stride < ff || (elem != 2 && elem != 4)) return B200KV_E_SHAPE;
-  const int vec = ff % 4 == 0 && stride % 4 == 0 && out_stride % 4 == 0 && aligned(gate_up, 16) && aligned(out, 16);
-  const long long items = (long long)num_rows * (vec ? ff / 4 : ff), blocks = (items + kRowThreads - 1) / kRowThreads;
-  if (blocks > 0x7FFFFFF0ll) return B200KV_E_RANGE;
+  const bool vec = ff % 8 == 0 && stride % 8 == 0 && out_stride % 8 == 0 && aligned(gate_up, 16) && aligned(out, 16);
+  const dim3 grid(num_rows, (ff / (vec ? 8 : 1) + kRowThreads - 1) / kRowThreads);
   cudaStream_t s = (cudaStream_t)stream;
   if (elem == 2)
-    return launch_result(launch_chained(silu_mul_rows_kernel<uint16_t>, dim3((unsigned)blocks), dim3(kRowThreads), 0, s,
-                                        (const uint16_t*)gate_up, (long long)stride, (uint16_t*)out, (long long)out_stride, num_rows, ff, vec));
-  return launch_result(launch_chained(silu_mul_rows_kernel<float>, dim3((unsigned)blocks), dim3(kRowThreads), 0, s, (const float*)gate_up,
-                                      (long long)stride, (float*)out, (long long)out_stride, num_rows, ff, vec));
+    return launch_result(launch_chained(vec ? silu_mul_rows_kernel<uint16_t, 8> : silu_mul_rows_kernel<uint16_t, 1>, grid, dim3(kRowThreads), 0, s,
+                                        (const uint16_t*)gate_up, (long long)stride, (uint16_t*)out, (long long)out_stride, num_rows, ff));
+  return launch_result(launch_chained(vec ? silu_mul_rows_kernel<float, 8> : silu_mul_rows_kernel<float, 1>, grid, dim3(kRowThreads), 0, s,
+                                      (const float*)gate_up, (long long)stride, (float*)out, (long long)out_stride, num_rows, ff));
 }
 
 extern "C" int b200dec_gated_norm(const float* o, const void* gate, int64_t gate_stride, int32_t gate_first, int32_t elem,

@@ -492,16 +492,39 @@ def recurrence_decode(rec: Recurrence, st: RecurrentState, x, step, beta, rows: 
 
 
 @K._ranged
-def recurrence_prefill(rec: Recurrence, st: RecurrentState, x, step, beta, rows: Rows, out: torch.Tensor) -> None:
-    """The prompt portions' rows: convolution, then the state through every portion; out fp32 [N, heads * vdim]."""
-    K._require_cuda(x, out, st.state)
+def conv_rows(rec: Recurrence, st: RecurrentState, x, step, beta, rows: Rows) -> torch.Tensor:
+    """silu(convolution) of the prompt portions' rows, all channels."""
+    K._require_cuda(x, st.ring)
     r, i = _recurrence_args(rec, st, x, step, beta)
     e = rows.entries()
     conv = torch.empty(rows.num_rows, _round8(rec.channels), device=x.device, dtype=x.dtype)
+    rc = _lib_dec().b200dec_conv_rows(ctypes.byref(r), ctypes.byref(i), ctypes.byref(e), conv.data_ptr(), K.status_word(x.device).data_ptr(),
+                                      K._stream())
+    _lib.check(rc, "conv_rows")
+    return conv
+
+
+@K._ranged
+def recurrence_prefill(rec: Recurrence, st: RecurrentState, x, step, beta, rows: Rows, out: torch.Tensor, form: str | None = None) -> None:
+    """The prompt portions' rows: convolution, then the state through every portion; out fp32 [N, heads * vdim].  `form`: which
+    kernel carries the state ("scan" token by token, any sizes; "blocked", "chunked"); default: the fastest that applies."""
+    K._require_cuda(x, out, st.state)
+    conv = conv_rows(rec, st, x, step, beta, rows)
+    r, i = _recurrence_args(rec, st, x, step, beta)
+    e = rows.entries()
     lib, status = _lib_dec(), K.status_word(x.device).data_ptr()
-    _lib.check(lib.b200dec_conv_rows(ctypes.byref(r), ctypes.byref(i), ctypes.byref(e), conv.data_ptr(), status, K._stream()), "conv_rows")
-    _lib.check(lib.b200dec_recurrence_scan(ctypes.byref(r), ctypes.byref(i), conv.data_ptr(), ctypes.byref(e), out.data_ptr(), status,
-                                           K._stream()), "recurrence_scan")
+    nbytes = lib.b200dec_recurrence_blocked_workspace(ctypes.byref(r), ctypes.byref(e)) if rec.skip is None else 0
+    if form is None:
+        form = "blocked" if nbytes else ("chunked" if lib.b200dec_state_space_chunked_applies(ctypes.byref(r)) else "scan")
+    if form == "chunked":
+        rc = lib.b200dec_state_space_chunked(ctypes.byref(r), ctypes.byref(i), conv.data_ptr(), ctypes.byref(e), out.data_ptr(), status, K._stream())
+    elif form == "blocked":
+        ws = torch.empty(nbytes, dtype=torch.uint8, device=x.device)
+        rc = lib.b200dec_recurrence_blocked(ctypes.byref(r), ctypes.byref(i), conv.data_ptr(), ctypes.byref(e), out.data_ptr(), ws.data_ptr(),
+                                            nbytes, status, K._stream())
+    else:
+        rc = lib.b200dec_recurrence_scan(ctypes.byref(r), ctypes.byref(i), conv.data_ptr(), ctypes.byref(e), out.data_ptr(), status, K._stream())
+    _lib.check(rc, f"recurrence_{form}")
 
 
 @K._ranged

@@ -239,14 +239,15 @@ def rec_want(rec, a_log, x, step, beta):
 
 
 KINDS = ["delta", "state_space"]
-SIZES = [(4, 4, 32, 32, 4), (6, 3, 20, 28, 3), (2, 1, 128, 128, 4), (3, 1, 9, 7, 5), (1, 1, 64, 48, 1), (2, 2, 144, 264, 2), (2, 1, 260, 40, 3)]
+SIZES = [(4, 4, 32, 32, 4), (4, 2, 40, 24, 3), (2, 2, 8, 72, 4), (6, 3, 20, 28, 3), (2, 1, 128, 128, 4), (3, 1, 9, 7, 5), (1, 1, 64, 48, 1), (2, 2, 144, 264, 2), (2, 1, 260, 40, 3)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("kind", KINDS)
 @pytest.mark.parametrize("heads,groups,dim,vdim,taps", SIZES)
 @pytest.mark.parametrize("strong", [False, True])
-def test_recurrence_portions_and_decoding(heads, groups, dim, vdim, taps, kind, dtype, strong):
+@pytest.mark.parametrize("form", [None, "scan"])
+def test_recurrence_portions_and_decoding(heads, groups, dim, vdim, taps, kind, dtype, strong, form):
     """Three sequences in random slots, cut in different ways, prompts beside decoding entries; the slots start as nonsense."""
     from inference_engine_b200 import ops
 
@@ -271,7 +272,7 @@ def test_recurrence_portions_and_decoding(heads, groups, dim, vdim, taps, kind, 
         out = torch.empty(rows.num_rows, heads * vdim, device=DEV)
         ops.recurrence_decode(rec, st, x, step, beta, rows, out)
         if rows.seq_ids is not None:
-            ops.recurrence_prefill(rec, st, x, step, beta, rows, out)
+            ops.recurrence_prefill(rec, st, x, step, beta, rows, out, form)
         o = 0
         for e in live:
             close(out[o : o + chunks[e]].view(-1, heads, vdim), want[e][at[e] : at[e] + chunks[e]], dtype, f32=5e-5, b16=3e-2)
