@@ -211,10 +211,11 @@ int b200dec_recurrence_blocked(const b200dec_recurrence* rec, const b200dec_recu
                                const b200dec_entries* ent, float* out, void* workspace, size_t workspace_bytes, int32_t* status,
                                void* stream);
 /* The same for a state-space layer of a bf16 model (one decay per head, dim <= 128, sizes and offsets multiples of 8), sixteen
- * tokens at a time on the tensor cores; _applies: 1 where this form does. */
-int b200dec_state_space_chunked_applies(const b200dec_recurrence* rec);
+ * tokens at a time on the tensor cores; workspace 16-byte aligned, its size 0 where this form does not apply. */
+size_t b200dec_state_space_chunked_workspace(const b200dec_recurrence* rec);
 int b200dec_state_space_chunked(const b200dec_recurrence* rec, const b200dec_recurrence_in* in, const void* conv_out,
-                                const b200dec_entries* ent, float* out, int32_t* status, void* stream);
+                                const b200dec_entries* ent, float* out, void* workspace, size_t workspace_bytes, int32_t sm_count,
+                                int32_t* status, void* stream);
 /* out[r] (element size elem) = out_scale * norm(o[r] (* silu(gate)  if gate_first)) * weight (* sigmoid(gate) otherwise), the norm
  * taken over `parts` equal parts of the row of `len` each by itself; weight fp32 [weight_len], repeated.  */
 int b200dec_gated_norm(const float* o, const void* gate, int64_t gate_stride, int32_t gate_first, int32_t elem, const float* weight,

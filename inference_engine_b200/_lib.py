@@ -158,8 +158,8 @@ DECODER_SIGNATURES = {
     "b200dec_recurrence_scan": (c_int32, [P_REC, P_REC_IN, c_void_p, P_ENT, c_void_p, c_void_p, c_void_p]),
     "b200dec_recurrence_blocked_workspace": (c_size_t, [P_REC, P_ENT]),
     "b200dec_recurrence_blocked": (c_int32, [P_REC, P_REC_IN, c_void_p, P_ENT, c_void_p, c_void_p, c_size_t, c_void_p, c_void_p]),
-    "b200dec_state_space_chunked_applies": (c_int32, [P_REC]),
-    "b200dec_state_space_chunked": (c_int32, [P_REC, P_REC_IN, c_void_p, P_ENT, c_void_p, c_void_p, c_void_p]),
+    "b200dec_state_space_chunked_workspace": (c_size_t, [P_REC]),
+    "b200dec_state_space_chunked": (c_int32, [P_REC, P_REC_IN, c_void_p, P_ENT, c_void_p, c_void_p, c_size_t, c_int32, c_void_p, c_void_p]),
     "b200dec_gated_norm": (c_int32, [c_void_p, c_void_p, c_int64, c_int32, c_int32, c_void_p, c_int32, c_float, c_float, c_void_p, c_int64,
                                      c_int32, c_int32, c_int32, c_void_p]),
     "b200dec_router": (c_int32, [c_void_p, c_void_p, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p, c_void_p, c_void_p,

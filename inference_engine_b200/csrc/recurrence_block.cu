@@ -195,14 +195,15 @@ __device__ __forceinline__ void rb_bulk(uint32_t dst, const void* src, uint32_t 
                ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
 
-// Sums of 32 values (token * 4 + column) over kLanes lanes, of which each keeps 32 / kLanes: those of token lane / (kLanes / 8)
-// and of column 4 / (kLanes / 8) * (lane % (kLanes / 8)) on.
+// Sums of 32 values over kLanes lanes, of which each keeps 32 / kLanes: those of token lane / (kLanes / 8) and of column
+// 4 / (kLanes / 8) * (lane % (kLanes / 8)) on.  A lane holds token i ^ (the token it will keep) in places 4 i .., so that what
+// it gives away in the exchanges over tokens always stands in the same places.
 template <int kLanes>
 __device__ __forceinline__ void rb_exchange(float (&v)[32], int lane) {
   int n = 16;
 #pragma unroll
   for (int bit = kLanes / 2; bit > 0; bit >>= 1) {
-    const bool hi = lane & bit;
+    const bool hi = n < 4 && (lane & bit);
 #pragma unroll
     for (int i = 0; i < n; ++i) {
       const float keep = hi ? v[i + n] : v[i], give = hi ? v[i] : v[i + n];
@@ -261,19 +262,20 @@ rb_scan_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, con
     S[2][i] = rb_pack(a.z, c.z);
     S[3][i] = rb_pack(a.w, c.w);
   }
-  auto value = [&](int b, float (&v)[kC]) {  // of this lane's token and columns in block b
+  // v of this lane's token and columns in block b; kept as loaded until it is used, so that nothing waits for it
+  auto value = [&](int b, T (&v)[kC]) {
     const int t = b * kRbTok + tok;
     const T* src = conv + (long long)(x.first + t) * conv_stride + rec.off_v + h * P + pc;
 #pragma unroll
-    for (int c = 0; c < kC; ++c) v[c] = t < x.n && pc + c < P ? ld_elem(src + c) : 0.f;
+    for (int c = 0; c < kC; ++c) v[c] = t < x.n && pc + c < P ? src[c] : T(0);
   };
-  float v_next[kC];
+  T v_next[kC];
   value(0, v_next);
   bool dead = false;
   for (int b = 0; b < blocks; ++b) {
     float w[kC];
 #pragma unroll
-    for (int c = 0; c < kC; ++c) w[c] = v_next[c];
+    for (int c = 0; c < kC; ++c) w[c] = ld_elem(v_next + c);
     value(b + 1, v_next);
     if (!dt_mbar_wait(dt_smem(bars + b % kRbStages), (b / kRbStages) & 1)) dead = true;
     const float* st = rb_smem + (b % kRbStages) * kFloats;
@@ -284,7 +286,7 @@ rb_scan_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, con
         rb_pair acc[4];
 #pragma unroll
         for (int j = 0; j < kQuads; ++j) {
-          const ulonglong2 k = reinterpret_cast<const ulonglong2*>(vec + i * Dp)[l + j * kLanes];
+          const ulonglong2 k = reinterpret_cast<const ulonglong2*>(vec + (i ^ tok) * Dp)[l + j * kLanes];
 #pragma unroll
           for (int c = 0; c < 4; ++c) {
             acc[c] = j == 0 ? rb_mul(S[c][0], k.x) : rb_fma(S[c][2 * j], k.x, acc[c]);
@@ -405,6 +407,8 @@ static int rb_run(const b200dec_recurrence& rec, const b200dec_recurrence_in& in
                   int32_t* status, cudaStream_t s) {
   if (rec.dim <= 32) return rb_launch<T, 8, 4>(rec, in, conv, ent, ws, out, status, s);
   if (rec.dim <= 64) return rb_launch<T, 16, 4>(rec, in, conv, ent, ws, out, status, s);
+  // few heads: more warps with fewer rows each, which is shorter per block and costs more in all
+  if (rec.dim <= 128 && (long long)rec.heads * ((rec.vdim + 15) / 16) < 256) return rb_launch<T, 32, 4>(rec, in, conv, ent, ws, out, status, s);
   if (rec.dim <= 128) return rb_launch<T, 16, 8>(rec, in, conv, ent, ws, out, status, s);
   return rb_launch<T, 32, 8>(rec, in, conv, ent, ws, out, status, s);
 }

@@ -513,17 +513,19 @@ def recurrence_prefill(rec: Recurrence, st: RecurrentState, x, step, beta, rows:
     r, i = _recurrence_args(rec, st, x, step, beta)
     e = rows.entries()
     lib, status = _lib_dec(), K.status_word(x.device).data_ptr()
-    nbytes = lib.b200dec_recurrence_blocked_workspace(ctypes.byref(r), ctypes.byref(e)) if rec.skip is None else 0
+    sizes = {"chunked": lib.b200dec_state_space_chunked_workspace(ctypes.byref(r)),
+             "blocked": lib.b200dec_recurrence_blocked_workspace(ctypes.byref(r), ctypes.byref(e)) if rec.skip is None else 0}
     if form is None:
-        form = "blocked" if nbytes else ("chunked" if lib.b200dec_state_space_chunked_applies(ctypes.byref(r)) else "scan")
-    if form == "chunked":
-        rc = lib.b200dec_state_space_chunked(ctypes.byref(r), ctypes.byref(i), conv.data_ptr(), ctypes.byref(e), out.data_ptr(), status, K._stream())
-    elif form == "blocked":
-        ws = torch.empty(nbytes, dtype=torch.uint8, device=x.device)
-        rc = lib.b200dec_recurrence_blocked(ctypes.byref(r), ctypes.byref(i), conv.data_ptr(), ctypes.byref(e), out.data_ptr(), ws.data_ptr(),
-                                            nbytes, status, K._stream())
-    else:
+        form = next((f for f, n in sizes.items() if n), "scan")
+    if form == "scan":
         rc = lib.b200dec_recurrence_scan(ctypes.byref(r), ctypes.byref(i), conv.data_ptr(), ctypes.byref(e), out.data_ptr(), status, K._stream())
+    else:
+        ws = torch.empty(sizes[form], dtype=torch.uint8, device=x.device)
+        args = (ctypes.byref(r), ctypes.byref(i), conv.data_ptr(), ctypes.byref(e), out.data_ptr(), ws.data_ptr(), sizes[form])
+        if form == "chunked":
+            rc = lib.b200dec_state_space_chunked(*args, K.num_sms(x.device), status, K._stream())
+        else:
+            rc = lib.b200dec_recurrence_blocked(*args, status, K._stream())
     _lib.check(rc, f"recurrence_{form}")
 
 

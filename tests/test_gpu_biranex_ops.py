@@ -283,6 +283,34 @@ def test_recurrence_portions_and_decoding(heads, groups, dim, vdim, taps, kind, 
     status_clear()
 
 
+@pytest.mark.parametrize("kind", KINDS)
+@pytest.mark.parametrize("heads,groups,dim,vdim", [(2, 1, 64, 64), (16, 4, 128, 72), (40, 8, 16, 16), (100, 4, 32, 8)])
+def test_long_portions_beside_others(kind, heads, groups, dim, vdim):
+    """Portions long enough to be cut into pieces that run side by side: one alone, two in a step, three beside a decoding one."""
+    from inference_engine_b200 import ops
+
+    g = np.random.default_rng(heads)
+    dtype = torch.bfloat16
+    rec, a_log = make_rec(g, kind, heads, groups, dim, vdim, 4)
+    st = ops.make_recurrent_state(rec, 4, dtype, DEV)
+    seqs = [rec_inputs(g, rec, 400, dtype) for _ in range(4)]
+    want = [rec_want(rec, a_log, *s) for s in seqs]
+    at = [0] * 4
+    for chunks in ([257, 0, 0, 0], [0, 129, 150, 0], [1, 64, 130, 200]):
+        live = [e for e in range(4) if chunks[e]]
+        rows, _ = step_rows([at[e] for e in live], [chunks[e] for e in live], int(chunks[0] == 1), slots=live)
+        x, step, beta = (None if i == 2 and not rec.correct else torch.cat([seqs[e][i][at[e] : at[e] + chunks[e]] for e in live]) for i in range(3))
+        out = torch.empty(rows.num_rows, heads * vdim, device=DEV)
+        ops.recurrence_decode(rec, st, x, step, beta, rows, out)
+        ops.recurrence_prefill(rec, st, x, step, beta, rows, out)
+        o = 0
+        for e in live:
+            close(out[o : o + chunks[e]].view(-1, heads, vdim), want[e][at[e] : at[e] + chunks[e]], dtype, b16=3e-2)
+            o += chunks[e]
+            at[e] += chunks[e]
+    status_clear()
+
+
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_decode_with_the_gated_norm_inside(dtype):
     from inference_engine_b200 import ops
