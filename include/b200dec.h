@@ -193,10 +193,11 @@ typedef struct b200dec_entries {
 
 /* The first *num_decoding rows, convolution and state in one kernel.  norm_w NULL: out fp32 [rows, heads * vdim] = o.
  * Otherwise out (element size elem, row stride out_stride) = o / sqrt(mean over vdim(o^2) + eps) * norm_w[vdim] *
- * sigmoid(gate) with gate rows [heads * vdim].  Rows from *num_decoding on of a pure decode step are zeroed. */
+ * sigmoid(gate) with gate rows [heads * vdim].  Rows from *num_decoding on of a pure decode step are zeroed.
+ * variant 0: states pass through shared memory on a persistent grid where they fit it (else as 1); 1: any size. */
 int b200dec_recurrence_decode(const b200dec_recurrence* rec, const b200dec_recurrence_in* in, const b200dec_entries* ent,
                               const float* norm_w, float eps, const void* gate, int64_t gate_stride, void* out, int64_t out_stride,
-                              int32_t* status, void* stream);
+                              int32_t variant, int32_t sm_count, int32_t* status, void* stream);
 /* Rows from *num_decoding on: silu(convolution) of every channel, conv_out [rows, channels rounded up to 8]. */
 int b200dec_conv_rows(const b200dec_recurrence* rec, const b200dec_recurrence_in* in, const b200dec_entries* ent, void* conv_out,
                       int32_t* status, void* stream);

@@ -152,8 +152,8 @@ DECODER_SIGNATURES = {
                                           c_int32, c_int32, c_void_p, c_void_p, c_void_p]),
     "b200dec_norm_add": (c_int32, [c_void_p, c_void_p, c_int32, c_void_p, c_float, c_float, c_void_p, c_int32, c_int32, c_void_p]),
     "b200dec_silu_mul": (c_int32, [c_void_p, c_int64, c_int32, c_void_p, c_int64, c_int32, c_int32, c_void_p]),
-    "b200dec_recurrence_decode": (c_int32, [P_REC, P_REC_IN, P_ENT, c_void_p, c_float, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
-                                            c_void_p]),
+    "b200dec_recurrence_decode": (c_int32, [P_REC, P_REC_IN, P_ENT, c_void_p, c_float, c_void_p, c_int64, c_void_p, c_int64, c_int32,
+                                            c_int32, c_void_p, c_void_p]),
     "b200dec_conv_rows": (c_int32, [P_REC, P_REC_IN, P_ENT, c_void_p, c_void_p, c_void_p]),
     "b200dec_recurrence_scan": (c_int32, [P_REC, P_REC_IN, c_void_p, P_ENT, c_void_p, c_void_p, c_void_p]),
     "b200dec_recurrence_blocked_workspace": (c_size_t, [P_REC, P_ENT]),

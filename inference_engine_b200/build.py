@@ -43,6 +43,7 @@ UNITS = {  # unit -> extra flags
     "moe.cu": [],
     "moe_gemm_tc5.cu": [],
     "recurrence.cu": [],
+    "recurrence_decode.cu": [],
     "recurrence_block.cu": [],
     "ssd_scan.cu": [],
 }
@@ -51,7 +52,7 @@ LIBRARIES = {
     LIB: ["abi.cu", "write_kernels.cu", "decode_attn.cu", "prefill_attn.cu", "prefill_attn_tc5.cu", "block_ops.cu", "sampler.cu",
           "skinny_linear_tc5.cu"],
     DECODER_LIB: ["abi.cu", "sampler.cu", "paged_prefill_tc5.cu", "row_ops.cu", "paged_rows.cu", "paged_decode.cu", "moe.cu", "moe_gemm_tc5.cu",
-                  "recurrence.cu", "recurrence_block.cu", "ssd_scan.cu"],
+                  "recurrence.cu", "recurrence_decode.cu", "recurrence_block.cu", "ssd_scan.cu"],
 }
 # The same library with per-warp timestamps compiled into the decode-attention kernel (bench.py --phases);
 # never loaded by the product path.

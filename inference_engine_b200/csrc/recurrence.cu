@@ -3,7 +3,7 @@
 // behind a short causal convolution per channel with silu.  o comes from the decayed state before the write:
 // o = (decay S)^T q + (k . q) u, so the two reductions over dim are made in one pass.
 //   decode  one block per (entry, head): convolution, norms, decays, state and (optionally) the gated output norm in one
-//           kernel.  HBM-bound: the state is read once and written once.
+//           kernel, for states of any size (recurrence_decode.cu has the one for the usual sizes).
 //   conv    prompt portions: silu(convolution) of every channel.
 //   scan    prompt portions, token after token, the state in registers: any sizes, both precisions.
 // The convolution's last inputs are kept by position modulo taps: a token writes the place that no token of its own
@@ -13,13 +13,6 @@
 namespace b200kv {
 
 constexpr int kRdThreads = 256;
-
-struct RecNorm {  // the output norm of the decode kernel
-  const float* weight;  // [vdim]; NULL: raw fp32 output
-  const void* gate;
-  long long gate_stride, out_stride;
-  float eps;
-};
 
 // Sum over the block; every thread gets it.
 __device__ __forceinline__ float rd_sum(float v, float* part) {
@@ -34,9 +27,9 @@ __device__ __forceinline__ float rd_sum(float v, float* part) {
 }
 
 // Threads are laid out as `rg` groups of rows by `cg` columns of four state entries; a thread owns rows r, r + rg, ...
-// kRows > 0: its entries stay in registers between the reduction and the update; 0: any size, the state is read twice.
-template <typename T, int kRows>
-__global__ void __launch_bounds__(kRdThreads, kRows <= 4 ? 4 : (kRows <= 8 ? 3 : 2))
+// The state is read twice, for the reduction and for the update, so that it may have any size.
+template <typename T>
+__global__ void __launch_bounds__(kRdThreads)
 recurrence_decode_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, const b200dec_entries ent, const RecNorm norm,
                          void* __restrict__ out, int cg, int rg, int32_t* status) {
   extern __shared__ __align__(16) float rd_smem[];
@@ -67,15 +60,6 @@ recurrence_decode_kernel(const b200dec_recurrence rec, const b200dec_recurrence_
   const int c4 = tid % cg, r0 = tid / cg;
   const bool mine = r0 < rg;
   float* state = rec.state + ((long long)x.slot * rec.heads + h) * D * P4;
-  float4 S[kRows > 0 ? kRows : 1];
-  if (kRows > 0) {
-#pragma unroll
-    for (int i = 0; i < kRows; ++i) {
-      const int d = r0 + i * rg;
-      S[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-      if (mine && d < D && x.pos > 0) S[i] = __ldcg(reinterpret_cast<const float4*>(state + (long long)d * P4) + c4);
-    }
-  }
   // ---- the token's q, k, v (convolution and silu), decays and step; two channels per thread at a time, all loads of
   // both ahead of the arithmetic
   const int per = rec.heads / rec.qk_heads, hq = h / per;
@@ -189,11 +173,7 @@ recurrence_decode_kernel(const b200dec_recurrence rec, const b200dec_recurrence_
       aq.x = fmaf(s.x, q, aq.x); aq.y = fmaf(s.y, q, aq.y); aq.z = fmaf(s.z, q, aq.z); aq.w = fmaf(s.w, q, aq.w);
     };
     if (in_row) {
-      if (kRows > 0) {
-#pragma unroll
-        for (int i = 0; i < kRows; ++i)
-          if (r0 + i * rg < D) add(S[i], r0 + i * rg);
-      } else if (x.pos > 0) {
+      if (x.pos > 0) {
         for (int d = r0; d < D; d += rg) {
           float4 s = __ldcg(reinterpret_cast<const float4*>(state + (long long)d * P4 + col));
           add(s, d);
@@ -225,18 +205,12 @@ recurrence_decode_kernel(const b200dec_recurrence rec, const b200dec_recurrence_
         s.x = fmaf(k, u.x, s.x); s.y = fmaf(k, u.y, s.y); s.z = fmaf(k, u.z, s.z); s.w = fmaf(k, u.w, s.w);
         *reinterpret_cast<float4*>(state + (long long)d * P4 + col) = s;
       };
-      if (kRows > 0) {
-#pragma unroll
-        for (int i = 0; i < kRows; ++i)
-          if (r0 + i * rg < D) move(S[i], r0 + i * rg);
-      } else {
-        for (int d = r0; d < D; d += rg) {
-          float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-          if (x.pos > 0) s = __ldcg(reinterpret_cast<const float4*>(state + (long long)d * P4 + col));
-          const float g = gs[d];
-          s.x *= g; s.y *= g; s.z *= g; s.w *= g;
-          move(s, d);
-        }
+      for (int d = r0; d < D; d += rg) {
+        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (x.pos > 0) s = __ldcg(reinterpret_cast<const float4*>(state + (long long)d * P4 + col));
+        const float g = gs[d];
+        s.x *= g; s.y *= g; s.z *= g; s.w *= g;
+        move(s, d);
       }
     }
   }
@@ -466,26 +440,21 @@ recurrence_scan_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in
   rec_keep_inputs<T>(rec, in, x, blockIdx.x, gridDim.x, kRsThreads);
 }
 
-template <typename T, int kRows>
-static int rd_launch(const b200dec_recurrence& rec, const b200dec_recurrence_in& in, const b200dec_entries& ent, const RecNorm& norm, void* out,
-                     int cg, int rg, int32_t* status, cudaStream_t s) {
-  const size_t smem = (size_t)(3 * rec_round4(rec.dim) + 3 * rec_round4(rec.vdim) + 8 * rg * cg) * 4;
-  if (smem > 200 * 1024) return B200KV_E_RANGE;
-  if (cudaFuncSetAttribute(recurrence_decode_kernel<T, kRows>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
-    return B200KV_E_LAUNCH;
-  return launch_result(launch_chained(recurrence_decode_kernel<T, kRows>, dim3(rec.heads, ent.num_entries), dim3(kRdThreads), smem, s, rec, in,
-                                      ent, norm, out, cg, rg, status));
-}
-
 template <typename T>
 static int rd_run(const b200dec_recurrence& rec, const b200dec_recurrence_in& in, const b200dec_entries& ent, const RecNorm& norm, void* out,
                   int32_t* status, cudaStream_t s) {
   const int quads = rec_round4(rec.vdim) / 4, cg = quads < kRdThreads ? quads : kRdThreads, rg = kRdThreads / cg;
-  const int rows = (rec.dim + rg - 1) / rg;
-  if (quads <= kRdThreads && rows <= 4) return rd_launch<T, 4>(rec, in, ent, norm, out, cg, rg, status, s);
-  if (quads <= kRdThreads && rows <= 8) return rd_launch<T, 8>(rec, in, ent, norm, out, cg, rg, status, s);
-  if (quads <= kRdThreads && rows <= 16) return rd_launch<T, 16>(rec, in, ent, norm, out, cg, rg, status, s);
-  return rd_launch<T, 0>(rec, in, ent, norm, out, cg, rg, status, s);
+  const size_t smem = (size_t)(3 * rec_round4(rec.dim) + 3 * rec_round4(rec.vdim) + 8 * rg * cg) * 4;
+  if (smem > 200 * 1024) return B200KV_E_RANGE;
+  if (cudaFuncSetAttribute(recurrence_decode_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    return B200KV_E_LAUNCH;
+  return launch_result(launch_chained(recurrence_decode_kernel<T>, dim3(rec.heads, ent.num_entries), dim3(kRdThreads), smem, s, rec, in, ent, norm,
+                                      out, cg, rg, status));
+}
+
+int recurrence_decode_any(const b200dec_recurrence& rec, const b200dec_recurrence_in& in, const b200dec_entries& ent, const RecNorm& norm,
+                          void* out, int32_t* status, cudaStream_t s) {
+  return rec.elem == 2 ? rd_run<uint16_t>(rec, in, ent, norm, out, status, s) : rd_run<float>(rec, in, ent, norm, out, status, s);
 }
 
 template <typename T, int kRows, int kLanes>
@@ -529,18 +498,6 @@ static int rc_run(const b200dec_recurrence& rec, const b200dec_recurrence_in& in
 }  // namespace b200kv
 
 using namespace b200kv;
-
-extern "C" int b200dec_recurrence_decode(const b200dec_recurrence* rec, const b200dec_recurrence_in* in, const b200dec_entries* ent,
-                                         const float* norm_w, float eps, const void* gate, int64_t gate_stride, void* out,
-                                         int64_t out_stride, int32_t* status, void* stream) {
-  const int rc = check_recurrence(rec, in, ent);
-  if (rc != B200KV_OK) return rc;
-  if (ent->num_entries == 0) return B200KV_OK;
-  if (!out || (norm_w && !gate)) return B200KV_E_NULL;
-  const RecNorm norm{norm_w, gate, gate_stride, out_stride, eps};
-  cudaStream_t s = (cudaStream_t)stream;
-  return rec->elem == 2 ? rd_run<uint16_t>(*rec, *in, *ent, norm, out, status, s) : rd_run<float>(*rec, *in, *ent, norm, out, status, s);
-}
 
 extern "C" int b200dec_conv_rows(const b200dec_recurrence* rec, const b200dec_recurrence_in* in, const b200dec_entries* ent, void* conv_out,
                                  int32_t* status, void* stream) {

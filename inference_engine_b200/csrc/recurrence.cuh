@@ -26,6 +26,13 @@ __device__ __forceinline__ RecEntry rec_entry(const b200dec_entries& ent, const 
   return x;
 }
 
+struct RecNorm {  // the output norm of the decode kernel
+  const float* weight;  // [vdim]; NULL: raw fp32 output
+  const void* gate;
+  long long gate_stride, out_stride;
+  float eps;
+};
+
 __host__ __device__ constexpr int rec_round4(int n) { return (n + 3) / 4 * 4; }
 
 __device__ __forceinline__ float ldcg_elem(const uint16_t* p) { return bf16_bits_to_float(__ldcg(p)); }

@@ -479,7 +479,7 @@ def _recurrence_args(rec: Recurrence, st: RecurrentState, x, step, beta):
 
 @K._ranged
 def recurrence_decode(rec: Recurrence, st: RecurrentState, x, step, beta, rows: Rows, out: torch.Tensor, norm: GatedNorm | None = None,
-                      gate: torch.Tensor | None = None) -> None:
+                      gate: torch.Tensor | None = None, variant: int = 0) -> None:
     """One token of every decoding entry: convolution, state and read-out; out fp32 [N, heads * vdim], or with `norm` (one part
     per head, gate behind it) the gated output in the model's precision."""
     K._require_cuda(x, out, st.state)
@@ -487,7 +487,8 @@ def recurrence_decode(rec: Recurrence, st: RecurrentState, x, step, beta, rows: 
     e = rows.entries()
     rc = _lib_dec().b200dec_recurrence_decode(
         ctypes.byref(r), ctypes.byref(i), ctypes.byref(e), None if norm is None else norm.weight.data_ptr(), 0.0 if norm is None else norm.eps,
-        _ptr(gate), 0 if gate is None else gate.stride(0), out.data_ptr(), out.stride(0), K.status_word(x.device).data_ptr(), K._stream())
+        _ptr(gate), 0 if gate is None else gate.stride(0), out.data_ptr(), out.stride(0), variant, K.num_sms(x.device),
+        K.status_word(x.device).data_ptr(), K._stream())
     _lib.check(rc, "recurrence_decode")
 
 
