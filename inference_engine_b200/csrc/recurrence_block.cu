@@ -17,6 +17,7 @@ namespace b200kv {
 
 constexpr int kRbTok = 8;        // tokens per block
 constexpr int kRbWarps = 2;      // of a block of the scan
+constexpr int kRbCols = 4;       // state columns of a group of lanes
 constexpr int kRbStages = 3;
 
 // Workspace of one (block, head) in floats: kd, qd, kr [8][Dp], L_8 [Dp], T [8][8], B [8][8].
@@ -26,19 +27,18 @@ __host__ __device__ constexpr int rb_floats(int Dp) { return 3 * kRbTok * Dp + D
 __device__ __forceinline__ int rb_first(const b200dec_entries& ent, int e) { return ent.cu_seqlens[e] / kRbTok + e; }
 
 // ---------------------------------------------------------------- prepare
-constexpr int kRpThreads = 256;
-constexpr int kRpChannels = 128;  // the first half of the threads sums A and the squares of k, the second B and those of q
-constexpr int kRpSums = 48;       // per half, padded for the exchange
+constexpr int kRpThreads = 128;
+constexpr int kRpSums = 96;  // A (28), B (36), squares of q and of k (8 each), padded for the exchange
 
-__host__ __device__ constexpr int rp_a(int i, int j) { return i * (i - 1) / 2 + j; }  // j < i: 28 sums
-__host__ __device__ constexpr int rp_b(int i, int j) { return i * (i + 1) / 2 + j; }  // j <= i: 36 sums
-constexpr int kRpSquares = 36;                                                          // 8 sums, in both halves
+__host__ __device__ constexpr int rp_a(int i, int j) { return i * (i - 1) / 2 + j; }       // j < i
+__host__ __device__ constexpr int rp_b(int i, int j) { return 28 + i * (i + 1) / 2 + j; }  // j <= i
+constexpr int kRpQ = 64, kRpK = 72;
 
-// Sums of 48 values over the warp's lanes; every lane keeps three (lanes 2 i and 2 i + 1 the same).
+// Sums of 96 values over the warp's lanes; every lane keeps three.
 __device__ __forceinline__ void rp_exchange(float (&v)[kRpSums], int lane) {
   int n = kRpSums / 2;
 #pragma unroll
-  for (int bit = 16; bit > 1; bit >>= 1) {
+  for (int bit = 16; bit > 0; bit >>= 1) {
     const bool hi = lane & bit;
 #pragma unroll
     for (int i = 0; i < n; ++i) {
@@ -47,18 +47,16 @@ __device__ __forceinline__ void rp_exchange(float (&v)[kRpSums], int lane) {
     }
     n >>= 1;
   }
-#pragma unroll
-  for (int i = 0; i < kRpSums / 16; ++i) v[i] += __shfl_xor_sync(0xffffffffu, v[i], 1);
 }
 
-template <typename T, bool kOne>  // kOne: dim <= kRpChannels, a thread's channel stays in registers
-__global__ void __launch_bounds__(kRpThreads, 2)
+template <typename T, bool kOne>  // kOne: dim <= kRpThreads, a thread's channel stays in registers
+__global__ void __launch_bounds__(kRpThreads)
 rb_prepare_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, const T* __restrict__ conv, int conv_stride,
                   const b200dec_entries ent, float* __restrict__ ws, int Dp, int32_t* status) {
-  __shared__ float red[2][4][kRpSums];
-  __shared__ float sums[2][kRpSums], beta[kRbTok], fq[kRbTok], fk[kRbTok];
+  __shared__ float red[kRpThreads / 32][kRpSums];
+  __shared__ float sums[kRpSums], beta[kRbTok], fq[kRbTok], fk[kRbTok];
   pdl_enter();
-  const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, half = tid / kRpChannels, ht = tid % kRpChannels, lane = tid & 31;
+  const int s = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31;
   int lo = 0, hi = ent.num_entries;
   while (hi - lo > 1) {
     const int mid = (lo + hi) >> 1;
@@ -72,18 +70,22 @@ rb_prepare_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, 
   const int D = rec.dim, hq = h / (rec.heads / rec.qk_heads);
   const long long row0 = x.first + t0;
   const float na = rec.neg_a[h];
-  float q[kRbTok], k[kRbTok], g[kRbTok];  // q only in the second half
+  const T* steps = (const T*)in.step + row0 * in.step_stride + h * D;
+  const T* src = conv + row0 * conv_stride + hq * D;
+  if (tid < kRbTok) beta[tid] = tid < nt ? sigmoid_f(ld_elem((const T*)in.beta + (row0 + tid) * in.beta_stride + h)) : 0.f;
+  float q[kRbTok], k[kRbTok], g[kRbTok];
   auto load = [&](int d) {
+    const float bias = d < D ? rec.dt_bias[h * D + d] : 0.f;
+    const T *pq = src + rec.off_q + d, *pk = src + rec.off_k + d, *ps = steps + d;
 #pragma unroll
     for (int i = 0; i < kRbTok; ++i) {
-      q[i] = k[i] = 0.f;
-      g[i] = 0.f;
-      if (i < nt && d < D) {
-        const T* src = conv + (row0 + i) * conv_stride;
-        if (half) q[i] = ld_elem(src + rec.off_q + hq * D + d);
-        k[i] = ld_elem(src + rec.off_k + hq * D + d);
-        g[i] = ld_elem((const T*)in.step + (row0 + i) * in.step_stride + h * D + d) + rec.dt_bias[h * D + d];
-      }
+      const bool some = i < nt && d < D;
+      q[i] = some ? ld_elem(pq) : 0.f;
+      k[i] = some ? ld_elem(pk) : 0.f;
+      g[i] = some ? ld_elem(ps) + bias : 0.f;
+      pq += conv_stride;
+      pk += conv_stride;
+      ps += in.step_stride;
     }
 #pragma unroll
     for (int i = 0; i < kRbTok; ++i) g[i] = i < nt && d < D ? expf(na * softplus_f(g[i])) : 1.f;
@@ -91,80 +93,68 @@ rb_prepare_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, 
   float v[kRpSums];
 #pragma unroll
   for (int i = 0; i < kRpSums; ++i) v[i] = 0.f;
-  if (tid < kRbTok) beta[tid] = tid < nt ? sigmoid_f(ld_elem((const T*)in.beta + (row0 + tid) * in.beta_stride + h)) : 0.f;
-  for (int d = ht; d < Dp; d += kRpChannels) {
+  for (int d = tid; d < Dp; d += kRpThreads) {
     load(d);
 #pragma unroll
     for (int j = 0; j < kRbTok; ++j) {
       float f = k[j];  // k_j times the decays since
-      if (half) {
-        v[rp_b(j, j)] = fmaf(q[j], f, v[rp_b(j, j)]);
-        v[kRpSquares + j] = fmaf(q[j], q[j], v[kRpSquares + j]);
-      } else {
-        v[kRpSquares + j] = fmaf(k[j], k[j], v[kRpSquares + j]);
-      }
+      v[rp_b(j, j)] = fmaf(q[j], f, v[rp_b(j, j)]);
+      v[kRpQ + j] = fmaf(q[j], q[j], v[kRpQ + j]);
+      v[kRpK + j] = fmaf(f, f, v[kRpK + j]);
 #pragma unroll
       for (int i = j + 1; i < kRbTok; ++i) {
         f *= g[i];
-        if (half) v[rp_b(i, j)] = fmaf(q[i], f, v[rp_b(i, j)]);
-        else v[rp_a(i, j)] = fmaf(k[i], f, v[rp_a(i, j)]);
+        v[rp_a(i, j)] = fmaf(k[i], f, v[rp_a(i, j)]);
+        v[rp_b(i, j)] = fmaf(q[i], f, v[rp_b(i, j)]);
       }
     }
   }
   rp_exchange(v, lane);
   {
-    const int at = ((lane >> 4) & 1) * 24 + ((lane >> 3) & 1) * 12 + ((lane >> 2) & 1) * 6 + ((lane >> 1) & 1) * 3;
-    if (!(lane & 1))
+    const int at = ((lane >> 4) & 1) * 48 + ((lane >> 3) & 1) * 24 + ((lane >> 2) & 1) * 12 + ((lane >> 1) & 1) * 6 + (lane & 1) * 3;
 #pragma unroll
-      for (int i = 0; i < 3; ++i) red[half][ht >> 5][at + i] = v[i];
+    for (int i = 0; i < 3; ++i) red[tid >> 5][at + i] = v[i];
   }
   __syncthreads();
-  if (ht < kRpSums) sums[half][ht] = (red[half][0][ht] + red[half][1][ht]) + (red[half][2][ht] + red[half][3][ht]);
+  if (tid < kRpSums) sums[tid] = (red[0][tid] + red[1][tid]) + (red[2][tid] + red[3][tid]);
   __syncthreads();
   if (tid < kRbTok) {
-    fq[tid] = rec.q_scale * (rec.unit_norm ? 1.0f / sqrtf(sums[1][kRpSquares + tid] + rec.unit_eps) : 1.f);
-    fk[tid] = rec.unit_norm ? 1.0f / sqrtf(sums[0][kRpSquares + tid] + rec.unit_eps) : 1.f;
+    fq[tid] = rec.q_scale * (rec.unit_norm ? 1.0f / sqrtf(sums[kRpQ + tid] + rec.unit_eps) : 1.f);
+    fk[tid] = rec.unit_norm ? 1.0f / sqrtf(sums[kRpK + tid] + rec.unit_eps) : 1.f;
   }
   __syncthreads();
   float* dst = ws + ((long long)s * rec.heads + h) * rb_floats(Dp);
   float* tb = dst + 3 * kRbTok * Dp + Dp;
+  for (int d = tid; d < Dp; d += kRpThreads) {
+    if (!kOne) load(d);
+    float f = 1.f;
+#pragma unroll
+    for (int i = 0; i < kRbTok; ++i) {
+      f *= g[i];
+      dst[i * Dp + d] = k[i] * fk[i] * f;
+      dst[(kRbTok + i) * Dp + d] = q[i] * fq[i] * f;
+    }
+    dst[3 * kRbTok * Dp + d] = f;
+    f = 1.f;
+#pragma unroll
+    for (int i = kRbTok - 1; i >= 0; --i) {
+      dst[(2 * kRbTok + i) * Dp + d] = k[i] * fk[i] * f;
+      f *= g[i];
+    }
+  }
   if (tid < kRbTok) {  // column tid of the inverse
     float c[kRbTok];
 #pragma unroll
     for (int i = 0; i < kRbTok; ++i) {
       float a = i == tid ? 1.f : 0.f;
 #pragma unroll
-      for (int j = 0; j < i; ++j) a = fmaf(-sums[0][rp_a(i, j)] * fk[i] * fk[j], c[j], a);
+      for (int j = 0; j < i; ++j) a = fmaf(-sums[rp_a(i, j)] * fk[i] * fk[j], c[j], a);
       c[i] = beta[i] * a;
       tb[i * kRbTok + tid] = c[i];
     }
-  } else if (ht >= 64 && half) {
-    const int i = (ht - 64) / kRbTok, j = ht % kRbTok;
-    tb[kRbTok * kRbTok + ht - 64] = j <= i ? sums[1][i * (i + 1) / 2 + j] * fq[i] * fk[j] : 0.f;
-  }
-  for (int d = ht; d < Dp; d += kRpChannels) {
-    if (!kOne) load(d);
-    float f = 1.f;
-    if (half) {
-#pragma unroll
-      for (int i = 0; i < kRbTok; ++i) {
-        f *= g[i];
-        dst[(kRbTok + i) * Dp + d] = q[i] * fq[i] * f;
-      }
-      dst[3 * kRbTok * Dp + d] = f;
-    } else {
-#pragma unroll
-      for (int i = 0; i < kRbTok; ++i) {
-        f *= g[i];
-        dst[i * Dp + d] = k[i] * fk[i] * f;
-      }
-      f = 1.f;
-#pragma unroll
-      for (int i = kRbTok - 1; i >= 0; --i) {
-        dst[(2 * kRbTok + i) * Dp + d] = k[i] * fk[i] * f;
-        f *= g[i];
-      }
-    }
+  } else if (tid >= 64) {
+    const int i = (tid - 64) / kRbTok, j = tid % kRbTok;
+    tb[kRbTok * kRbTok + tid - 64] = j <= i ? sums[28 + i * (i + 1) / 2 + j] * fq[i] * fk[j] : 0.f;
   }
 }
 
@@ -190,20 +180,25 @@ __device__ __forceinline__ rb_pair rb_mul(rb_pair a, rb_pair b) {
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
   return r;
 }
+// Volatile, so that the loads stay in front of the arithmetic they feed instead of beside it.
+__device__ __forceinline__ ulonglong2 rb_lds(uint32_t addr) {
+  ulonglong2 v;
+  asm volatile("ld.shared.v2.u64 {%0, %1}, [%2];" : "=l"(v.x), "=l"(v.y) : "r"(addr));
+  return v;
+}
 __device__ __forceinline__ void rb_bulk(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
   asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];\n"
                ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
 
-// Sums of 32 values over kLanes lanes, of which each keeps 32 / kLanes: those of token lane / (kLanes / 8) and of column
-// 4 / (kLanes / 8) * (lane % (kLanes / 8)) on.  A lane holds token i ^ (the token it will keep) in places 4 i .., so that what
-// it gives away in the exchanges over tokens always stands in the same places.
+// Sums of 32 values over kLanes lanes, of which each keeps 32 / kLanes: those of token lane / (kLanes / 8) and of columns
+// kC * (lane % (kLanes / 8)) on, kC = 32 / kLanes.  A lane holds token i ^ (the token it will keep) in places 4 i .., so that what it gives away in the exchanges over tokens always stands in the same places.
 template <int kLanes>
-__device__ __forceinline__ void rb_exchange(float (&v)[32], int lane) {
-  int n = 16;
+__device__ __forceinline__ void rb_exchange(float (&v)[kRbCols * kRbTok], int lane) {
+  int n = kRbCols * kRbTok / 2;
 #pragma unroll
   for (int bit = kLanes / 2; bit > 0; bit >>= 1) {
-    const bool hi = n < 4 && (lane & bit);
+    const bool hi = n < kRbCols && (lane & bit);
 #pragma unroll
     for (int i = 0; i < n; ++i) {
       const float keep = hi ? v[i + n] : v[i], give = hi ? v[i] : v[i + n];
@@ -213,16 +208,16 @@ __device__ __forceinline__ void rb_exchange(float (&v)[32], int lane) {
   }
 }
 
-// kLanes lanes share four state columns; lane l owns rows 4 kLanes j + 4 l + (0..3), j < kR / 4, of all four.
-// One block: kRbWarps warps, 128 / kLanes columns each, of one head of one entry.
+// kLanes lanes share kRbCols state columns; lane l owns rows 4 kLanes j + 4 l + (0..3), j < kR / 4, of all of them.
+// One block: kRbWarps warps, 32 kRbCols / kLanes columns each, of one head of one entry.
 template <typename T, int kLanes, int kR>
 __global__ void __launch_bounds__(32 * kRbWarps)
 rb_scan_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, const T* __restrict__ conv, int conv_stride,
                const b200dec_entries ent, const float* __restrict__ ws, float* __restrict__ out, int slabs, int32_t* status) {
   constexpr int Dp = kLanes * kR, kFloats = rb_floats(Dp), kQuads = kR / 4, kGroups = 32 / kLanes;
-  constexpr int kM = kLanes / 8, kC = 4 / kM;  // after the exchange a lane holds kC columns of one token
+  constexpr int kM = kLanes / 8, kC = kRbCols / kM;  // after the exchange a lane holds kC columns of one token
   extern __shared__ __align__(128) float rb_smem[];  // [kRbStages][kFloats]
-  __shared__ __align__(16) float ubuf[kRbWarps][kGroups][kRbTok][4];
+  __shared__ __align__(16) float ubuf[kRbWarps][kGroups][kRbTok][kRbCols];
   __shared__ __align__(8) uint64_t bars[kRbStages];
   pdl_enter();
   const int e = blockIdx.y, h = blockIdx.x / slabs, slab = blockIdx.x - h * slabs, tid = threadIdx.x;
@@ -237,7 +232,7 @@ rb_scan_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, con
   if (x.n == 0) return;
   const int D = rec.dim, P = rec.vdim, P4 = rec_round4(P), blocks = (x.n + kRbTok - 1) / kRbTok;
   const int warp = tid >> 5, grp = (tid & 31) / kLanes, l = tid % kLanes;
-  const int p0 = (slab * kRbWarps + warp) * 4 * kGroups + 4 * grp;  // the four columns
+  const int p0 = ((slab * kRbWarps + warp) * kGroups + grp) * kRbCols;  // the first column
   const int tok = l / kM, pc = p0 + kC * (l % kM);                  // what this lane holds after the exchange
   const long long at0 = (long long)rb_first(ent, e) * rec.heads + h;
   auto fetch = [&](int b) {
@@ -248,7 +243,7 @@ rb_scan_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, con
   if (tid == 0)
     for (int b = 0; b < min(kRbStages, blocks); ++b) fetch(b);
   float* state = rec.state + ((long long)x.slot * rec.heads + h) * D * P4;
-  rb_pair S[4][kR / 2];  // [column][pair of rows]
+  rb_pair S[kRbCols][kR / 2];  // [column][pair of rows]
 #pragma unroll
   for (int i = 0; i < kR / 2; ++i) {
     const int d = (i / 2) * 4 * kLanes + 4 * l + 2 * (i & 1);
@@ -279,28 +274,42 @@ rb_scan_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, con
     value(b + 1, v_next);
     if (!dt_mbar_wait(dt_smem(bars + b % kRbStages), (b / kRbStages) & 1)) dead = true;
     const float* st = rb_smem + (b % kRbStages) * kFloats;
-    // sums over the rows of the state times eight vectors, exchanged
-    auto sums = [&](const float* vec, float (&r)[32]) {
+    // this lane's rows of eight vectors (of token i ^ swap in place i), and their sums with the state
+    const uint32_t mine = dt_smem(st) + 16 * l;
+    auto rows = [&](int vec, int swap, ulonglong2 (&k)[kRbTok][kQuads]) {
+#pragma unroll
+      for (int i = 0; i < kRbTok; ++i)
+#pragma unroll
+        for (int j = 0; j < kQuads; ++j) k[i][j] = rb_lds(mine + 4 * ((vec * kRbTok + (i ^ swap)) * Dp + 4 * kLanes * j));
+    };
+    auto sums = [&](const ulonglong2 (&vec)[kRbTok][kQuads], float (&r)[kRbCols * kRbTok]) {
 #pragma unroll
       for (int i = 0; i < kRbTok; ++i) {
-        rb_pair acc[4];
+        rb_pair acc[kRbCols];
 #pragma unroll
         for (int j = 0; j < kQuads; ++j) {
-          const ulonglong2 k = reinterpret_cast<const ulonglong2*>(vec + (i ^ tok) * Dp)[l + j * kLanes];
+          const ulonglong2 k = vec[i][j];
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
+          for (int c = 0; c < kRbCols; ++c) {
             acc[c] = j == 0 ? rb_mul(S[c][0], k.x) : rb_fma(S[c][2 * j], k.x, acc[c]);
             acc[c] = rb_fma(S[c][2 * j + 1], k.y, acc[c]);
           }
         }
 #pragma unroll
-        for (int c = 0; c < 4; ++c) r[4 * i + c] = rb_both(acc[c]);
+        for (int c = 0; c < kRbCols; ++c) r[kRbCols * i + c] = rb_both(acc[c]);
       }
-      rb_exchange<kLanes>(r, l);
     };
-    float r[32], o[32];
-    sums(st, r);
-    sums(st + kRbTok * Dp, o);
+    ulonglong2 ka[kRbTok][kQuads], kb[kRbTok][kQuads], decay[kQuads];
+    float r[kRbCols * kRbTok], o[kRbCols * kRbTok];
+    rows(0, tok, ka);
+    rows(1, tok, kb);
+    sums(ka, r);
+    rows(2, 0, ka);
+    rb_exchange<kLanes>(r, l);
+    sums(kb, o);
+#pragma unroll
+    for (int j = 0; j < kQuads; ++j) decay[j] = rb_lds(mine + 4 * (3 * kRbTok * Dp + 4 * kLanes * j));
+    rb_exchange<kLanes>(o, l);
     const float* tb = st + 3 * kRbTok * Dp + Dp;
     float row[2][kRbTok];
 #pragma unroll
@@ -337,9 +346,9 @@ rb_scan_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, con
     }
 #pragma unroll
     for (int j = 0; j < kQuads; ++j) {
-      const ulonglong2 g = reinterpret_cast<const ulonglong2*>(st + 3 * kRbTok * Dp)[l + j * kLanes];
+      const ulonglong2 g = decay[j];
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < kRbCols; ++c) {
         S[c][2 * j] = rb_mul(S[c][2 * j], g.x);
         S[c][2 * j + 1] = rb_mul(S[c][2 * j + 1], g.y);
       }
@@ -347,12 +356,12 @@ rb_scan_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, con
 #pragma unroll
     for (int i = 0; i < kRbTok; ++i) {
       const float4 uu = *reinterpret_cast<const float4*>(ubuf[warp][grp][i]);
-      const rb_pair up[4] = {rb_pack(uu.x, uu.x), rb_pack(uu.y, uu.y), rb_pack(uu.z, uu.z), rb_pack(uu.w, uu.w)};
+      const rb_pair up[kRbCols] = {rb_pack(uu.x, uu.x), rb_pack(uu.y, uu.y), rb_pack(uu.z, uu.z), rb_pack(uu.w, uu.w)};
 #pragma unroll
       for (int j = 0; j < kQuads; ++j) {
-        const ulonglong2 k = reinterpret_cast<const ulonglong2*>(st + (2 * kRbTok + i) * Dp)[l + j * kLanes];
+        const ulonglong2 k = ka[i][j];
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c < kRbCols; ++c) {
           S[c][2 * j] = rb_fma(k.x, up[c], S[c][2 * j]);
           S[c][2 * j + 1] = rb_fma(k.y, up[c], S[c][2 * j + 1]);
         }
@@ -371,9 +380,9 @@ rb_scan_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, con
 #pragma unroll
   for (int i = 0; i < kR / 2; ++i) {
     const int d = (i / 2) * 4 * kLanes + 4 * l + 2 * (i & 1);
-    float a[4], c[4];
+    float a[kRbCols], c[kRbCols];
 #pragma unroll
-    for (int k = 0; k < 4; ++k) {
+    for (int k = 0; k < kRbCols; ++k) {
       asm("mov.b64 {%0, %1}, %2;" : "=f"(a[k]), "=f"(c[k]) : "l"(S[k][i]));
       if (p0 + k >= P) a[k] = c[k] = 0.f;
     }
@@ -388,17 +397,19 @@ rb_scan_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in in, con
 template <typename T, int kLanes, int kR>
 static int rb_launch(const b200dec_recurrence& rec, const b200dec_recurrence_in& in, const void* conv, const b200dec_entries& ent, float* ws,
                      float* out, int32_t* status, cudaStream_t s) {
-  constexpr int Dp = kLanes * kR, kCols = kRbWarps * 128 / kLanes;
+  constexpr int Dp = kLanes * kR, kCols = kRbWarps * 32 / kLanes * kRbCols;
   const int stride = (rec.channels + 7) / 8 * 8, slabs = (rec.vdim + kCols - 1) / kCols;
   const int list = ent.num_rows / kRbTok + ent.num_entries;
-  auto* prepare = rec.dim <= kRpChannels ? rb_prepare_kernel<T, true> : rb_prepare_kernel<T, false>;
+  auto* prepare = rec.dim <= kRpThreads ? rb_prepare_kernel<T, true> : rb_prepare_kernel<T, false>;
   const int rc = launch_result(launch_chained(prepare, dim3(list, rec.heads), dim3(kRpThreads), 0, s, rec, in, (const T*)conv, stride, ent, ws, Dp,
                                               status));
   if (rc != B200KV_OK) return rc;
   const size_t smem = (size_t)kRbStages * rb_floats(Dp) * 4;
   if (cudaFuncSetAttribute(rb_scan_kernel<T, kLanes, kR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
     return B200KV_E_LAUNCH;
-  return launch_result(launch_chained(rb_scan_kernel<T, kLanes, kR>, dim3(rec.heads * slabs, ent.num_entries), dim3(32 * kRbWarps), smem, s, rec, in,
+  // Not chained: brought up beside the kernel in front, its few long-running blocks would crowd on the multiprocessors that
+  // come free first.
+  return launch_result(launch_kernel(false, rb_scan_kernel<T, kLanes, kR>, dim3(rec.heads * slabs, ent.num_entries), dim3(32 * kRbWarps), smem, s, rec, in,
                                       (const T*)conv, stride, ent, (const float*)ws, out, slabs, status));
 }
 
@@ -407,8 +418,6 @@ static int rb_run(const b200dec_recurrence& rec, const b200dec_recurrence_in& in
                   int32_t* status, cudaStream_t s) {
   if (rec.dim <= 32) return rb_launch<T, 8, 4>(rec, in, conv, ent, ws, out, status, s);
   if (rec.dim <= 64) return rb_launch<T, 16, 4>(rec, in, conv, ent, ws, out, status, s);
-  // few heads: more warps with fewer rows each, which is shorter per block and costs more in all
-  if (rec.dim <= 128 && (long long)rec.heads * ((rec.vdim + 15) / 16) < 256) return rb_launch<T, 32, 4>(rec, in, conv, ent, ws, out, status, s);
   if (rec.dim <= 128) return rb_launch<T, 16, 8>(rec, in, conv, ent, ws, out, status, s);
   return rb_launch<T, 32, 8>(rec, in, conv, ent, ws, out, status, s);
 }
