@@ -22,6 +22,24 @@ __device__ __forceinline__ void rpd_store(void* dst, uint32_t src, uint32_t byte
   asm volatile("cp.async.bulk.commit_group;\n" ::: "memory");
 }
 
+// Two neighbouring columns per instruction.
+typedef unsigned long long rpd_pair;
+__device__ __forceinline__ rpd_pair rpd_both(float a) {
+  rpd_pair r;
+  asm("mov.b64 %0, {%1, %1};" : "=l"(r) : "f"(a));
+  return r;
+}
+__device__ __forceinline__ rpd_pair rpd_mul(rpd_pair a, rpd_pair b) {
+  rpd_pair r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ rpd_pair rpd_fma(rpd_pair a, rpd_pair b, rpd_pair c) {
+  rpd_pair r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+
 // What an item needs beside its state: up to two channels per thread of q | k | v (dim, dim, vdim of them).  The items of a
 // group of heads follow one another; all but the first find q and k where the one before left them.
 template <typename T>
@@ -200,23 +218,26 @@ recurrence_step_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in
     }
     if (!dt_mbar_wait(dt_smem(bars + i % kRpdStages), (i / kRpdStages) & 1)) dead = true;
     float* st = stage(i);
-    float4 S[kRows];
+    ulonglong2 S[kRows];
     if (ok && !dead && mine) {
-      float4 ak = make_float4(0.f, 0.f, 0.f, 0.f), aq = ak;
+      ulonglong2 ak = make_ulonglong2(0ull, 0ull), aq = ak;
 #pragma unroll
       for (int j = 0; j < kRows; ++j) {
         const int d = r0 + j * rg;
         if (d >= D) break;
-        float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (!fresh) s = *reinterpret_cast<const float4*>(st + d * P4 + 4 * c4);
-        const float g = gs[d], k = ks[d], q = qs[d];
-        s.x *= g; s.y *= g; s.z *= g; s.w *= g;
-        ak.x = fmaf(s.x, k, ak.x); ak.y = fmaf(s.y, k, ak.y); ak.z = fmaf(s.z, k, ak.z); ak.w = fmaf(s.w, k, ak.w);
-        aq.x = fmaf(s.x, q, aq.x); aq.y = fmaf(s.y, q, aq.y); aq.z = fmaf(s.z, q, aq.z); aq.w = fmaf(s.w, q, aq.w);
+        ulonglong2 s = make_ulonglong2(0ull, 0ull);
+        if (!fresh) s = *reinterpret_cast<const ulonglong2*>(st + d * P4 + 4 * c4);
+        const rpd_pair g = rpd_both(gs[d]), k = rpd_both(ks[d]), q = rpd_both(qs[d]);
+        s.x = rpd_mul(s.x, g);
+        s.y = rpd_mul(s.y, g);
+        ak.x = rpd_fma(s.x, k, ak.x);
+        ak.y = rpd_fma(s.y, k, ak.y);
+        aq.x = rpd_fma(s.x, q, aq.x);
+        aq.y = rpd_fma(s.y, q, aq.y);
         S[j] = s;
       }
-      *reinterpret_cast<float4*>(red + r0 * 4 * cg + 4 * c4) = ak;
-      *reinterpret_cast<float4*>(red + (rg + r0) * 4 * cg + 4 * c4) = aq;
+      *reinterpret_cast<ulonglong2*>(red + r0 * 4 * cg + 4 * c4) = ak;
+      *reinterpret_cast<ulonglong2*>(red + (rg + r0) * 4 * cg + 4 * c4) = aq;
     }
     __syncthreads();
     float ss = 0.f;
@@ -249,15 +270,13 @@ recurrence_step_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in
     __syncthreads();
     if (norm.weight && (tid & 31) == 0) part[3][tid >> 5] = ss;
     if (ok && !dead && mine) {
-      const float4 u = *reinterpret_cast<const float4*>(us + 4 * c4);
+      const ulonglong2 u = *reinterpret_cast<const ulonglong2*>(us + 4 * c4);
 #pragma unroll
       for (int j = 0; j < kRows; ++j) {
         const int d = r0 + j * rg;
         if (d >= D) break;
-        const float k = ks[d];
-        float4 s = S[j];
-        s.x = fmaf(k, u.x, s.x); s.y = fmaf(k, u.y, s.y); s.z = fmaf(k, u.z, s.z); s.w = fmaf(k, u.w, s.w);
-        *reinterpret_cast<float4*>(st + d * P4 + 4 * c4) = s;
+        const rpd_pair k = rpd_both(ks[d]);
+        *reinterpret_cast<ulonglong2*>(st + d * P4 + 4 * c4) = make_ulonglong2(rpd_fma(k, u.x, S[j].x), rpd_fma(k, u.y, S[j].y));
       }
     }
     asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");  // the new state, for the copy out
