@@ -153,7 +153,8 @@ recurrence_step_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in
       }
     }
   };
-  if (tid == 0)
+  const bool copier = tid == kRpdThreads - 32;  // in a warp that has no columns to add up
+  if (copier)
     for (int i = 0; i < min(kRpdStages - 1, n); ++i) fetch(i);
   RpdItem<T> t;
   Where where = look(i0 / H, i0 % H);
@@ -209,6 +210,10 @@ recurrence_step_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in
     if (i + 1 < n) {
       gather(where, !ok, t);
       where = after(where);
+    }
+    if (copier && i + kRpdStages - 1 < n) {  // into the stage of the item before, once its copy out has been read
+      asm volatile("cp.async.bulk.wait_group.read 0;\n" ::: "memory");
+      fetch(i + kRpdStages - 1);
     }
     float qk = 0.f;
     if (ok && !same) {
@@ -282,22 +287,15 @@ recurrence_step_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in
     asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");  // the new state, for the copy out
     const bool stop = __syncthreads_or(dead);
     if (stop) {
-      if (tid == 0) {
+      if (copier) {
         if (status) atomicOr(status, B200KV_S_TIMEOUT);
-        for (int j = i; j < min(i + kRpdStages - 1, n); ++j) dt_mbar_wait(dt_smem(bars + j % kRpdStages), (j / kRpdStages) & 1);
+        for (int j = i; j < min(i + kRpdStages, n); ++j) dt_mbar_wait(dt_smem(bars + j % kRpdStages), (j / kRpdStages) & 1);
         asm volatile("cp.async.bulk.wait_group 0;\n" ::: "memory");
       }
       __syncthreads();
       return;
     }
-    if (tid == 0) {
-      if (ok) rpd_store(state_of(slot, h), dt_smem(st), bytes);
-      else asm volatile("cp.async.bulk.commit_group;\n" ::: "memory");
-      if (i + kRpdStages - 1 < n) {  // into the stage of the item before, whose copy out has been read by now
-        asm volatile("cp.async.bulk.wait_group.read 1;\n" ::: "memory");
-        fetch(i + kRpdStages - 1);
-      }
-    }
+    if (copier && ok) rpd_store(state_of(slot, h), dt_smem(st), bytes);
     if (norm.weight && ok) {
       float sum = 0.f;
 #pragma unroll
@@ -305,11 +303,10 @@ recurrence_step_kernel(const b200dec_recurrence rec, const b200dec_recurrence_in
       if (tid < P) {
         const float inv = 1.0f / sqrtf(sum / (float)P + norm.eps);
         st_elem((T*)out + row * norm.out_stride + h * P + tid, os[tid] * inv * norm_w * sigmoid_act<T>(gate));
-      }
-      __syncthreads();  // part and os are free
+      }  // os and part[3] are written again behind two barriers of the next item
     }
   }
-  if (tid == 0) asm volatile("cp.async.bulk.wait_group 0;\n" ::: "memory");
+  if (copier) asm volatile("cp.async.bulk.wait_group 0;\n" ::: "memory");
 }
 
 struct RpdShape {
